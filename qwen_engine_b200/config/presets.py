@@ -100,6 +100,23 @@ PRESETS: dict[str, dict[str, Any]] = {
                                             rot=dict(base=10000.0, dims=8, scaling=None)),
                                  mlp=None)]),
         init=dict(seed=17, std=0.08, norm_std=0.1, block_size=16)),
+    # a small model of the Zugunex design: latent attention with a sink, a gate per head and windows of 40 and 24 tokens,
+    # the second and third layers reading the first one's latent; a dense feed-forward and experts beside a shared one
+    "zugunex-tiny": dict(
+        config=dict(architecture="Zugunex", vocab=320, width=128, norm=dict(eps=1e-6),
+                    layers=[dict(type="latent_attention",
+                                 mixer=dict(heads=4, dim=32, rot_dim=16, vdim=24, kv_rank=48, scale=0.14, mask=dict(size=40),
+                                            rot=dict(base=20000.0, dims=16)),
+                                 mlp=dict(kind="dense", ff=256)),
+                            dict(type="latent_attention",
+                                 mixer=dict(heads=4, dim=32, rot_dim=16, vdim=24, kv_rank=48, scale=0.14, mask=dict(size=24),
+                                            rot=dict(base=20000.0, dims=16), kv_from=0),
+                                 mlp=dict(kind="moe", expert=dict(ff=64), router=dict(experts=4, top=2, scale=1.2), shared=dict(ff=96))),
+                            dict(type="latent_attention",
+                                 mixer=dict(heads=2, dim=16, rot_dim=16, vdim=32, kv_rank=48, scale=0.18, mask=dict(size=40),
+                                            rot=dict(base=20000.0, dims=16), kv_from=0),
+                                 mlp=None)]),
+        init=dict(seed=23, std=0.08, norm_std=0.1, block_size=16)),
 }
 
 

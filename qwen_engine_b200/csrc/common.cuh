@@ -63,6 +63,25 @@ __device__ __forceinline__ float gate_act_fast(float g, int act) {
   return __fdividef(g, 1.f + __expf(-g));
 }
 
+// The activation of a feed-forward without a gate, on the sums of its first product: 0 none, 1 the tanh form of gelu, 2 the
+// square of relu, 3 silu.  act_exact uses the library's tanh and exponential (float32 results), act_fast the hardware's
+// (bfloat16 results); the entry points of the products take the code in the bits of `out_mode` above the lowest one.
+__device__ __forceinline__ float act_exact(float z, int act) {
+  if (act == 0) return z;
+  if (act == 2) { const float r = fmaxf(z, 0.f); return r * r; }
+  if (act == 1) return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  return z / (1.f + expf(-z));
+}
+__device__ __forceinline__ float act_fast(float z, int act) {
+  if (act == 0) return z;
+  if (act == 2) { const float r = fmaxf(z, 0.f); return r * r; }
+  return gate_act_fast(z, act == 1 ? 1 : 0);
+}
+template <typename TOut> __device__ __forceinline__ float act_for(float z, int act) {
+  return sizeof(TOut) == 4 ? act_exact(z, act) : act_fast(z, act);
+}
+#define QE_ACT_MAX 3
+
 // A gated feed-forward's value from its gate g and its up projection u.  act 0 and 1: act(g) * u as above.  Any
 // other value of act is the bit pattern of a float32 limit L > 0 (every such pattern is an integer above 1) and
 // names the limited form: g' = min(g, L), u' = clamp(u, -L, L), g' * sigmoid(1.702 g') * (u' + 1).

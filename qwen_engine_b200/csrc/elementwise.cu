@@ -7,13 +7,14 @@
 
 // ---------------------------------------------------------------------------------------
 // out[t, :] = float(table[ids[t], :]) * scale   (reference src/layers/ops/embedding.py:28-44; scale 1 there),
-// or, with `accumulate`, out[t, :] += that (a pass that starts again from the tokens).
+// or, with `accumulate`, out[t, :] += that (a pass that starts again from the tokens).  `copy` (may be null) gets the rows
+// once more in the table's type.
 // The residual stream is float32 in both paths.  An id outside the table gives NaN rows.
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restrict__ table,
                                  float* __restrict__ out, int H, int V, float* __restrict__ ssq_out, int ssq_ld,
-                                 float scale, int accumulate) {
+                                 float scale, int accumulate, T* __restrict__ copy) {
   __shared__ float scratch[33];
   const int t = blockIdx.x;
   pdl_launch_dependents();
@@ -23,7 +24,10 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
   const int id = ids[t];
   float* dst = out + (size_t)t * H;
   if (id < 0 || id >= V) {
-    for (int h = threadIdx.x; h < H; h += blockDim.x) dst[h] = __int_as_float(0x7fc00000);
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+      dst[h] = __int_as_float(0x7fc00000);
+      if (copy) copy[(size_t)t * H + h] = from_f32<T>(__int_as_float(0x7fc00000));
+    }
     return;
   }
   const T* src = table + (size_t)id * H;
@@ -32,7 +36,7 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
     for (int h = threadIdx.x; h < H; h += blockDim.x) dst[h] += to_f32(src[h]) * scale;
     return;
   }
-  for (int h = threadIdx.x; h < H; h += blockDim.x) { const float v = to_f32(src[h]) * scale; dst[h] = v; ss += v * v; }
+  for (int h = threadIdx.x; h < H; h += blockDim.x) { const float v = to_f32(src[h]) * scale; dst[h] = v; ss += v * v; if (copy) copy[(size_t)t * H + h] = from_f32<T>(v); }
   if (ssq_out) {                                   // the row's sum of squares, for a norm fused downstream
     ss = block_sum(ss, scratch);
     if (threadIdx.x == 0) ssq_out[(size_t)t * ssq_ld] = ss;
@@ -40,15 +44,16 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
 }
 
 extern "C" int qe_embedding(const int* ids, const void* table, float* out, int T, int H, int V,
-                            int dtype, float* ssq_out, int ssq_ld, float scale, int accumulate, cudaStream_t stream) {
+                            int dtype, float* ssq_out, int ssq_ld, float scale, int accumulate, void* copy,
+                            cudaStream_t stream) {
   if (T <= 0) return 0;
   if (accumulate) ssq_out = nullptr;
   if (dtype == QE_DTYPE_F32)
     qe_launch(embedding_kernel<float>, dim3(T), dim3(256), 0, stream, ids, (const float*)table, out, H, V, ssq_out, ssq_ld,
-              scale, accumulate);
+              scale, accumulate, (float*)copy);
   else if (dtype == QE_DTYPE_BF16)
     qe_launch(embedding_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, stream, ids, (const __nv_bfloat16*)table, out, H, V, ssq_out,
-              ssq_ld, scale, accumulate);
+              ssq_ld, scale, accumulate, (__nv_bfloat16*)copy);
   else QE_REFUSE("embedding: unknown dtype %d", dtype);
   QE_CHECK_LAUNCH("embedding");
   return 0;

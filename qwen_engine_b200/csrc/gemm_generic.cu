@@ -14,7 +14,7 @@
 template <typename TIn, typename TOut>
 __global__ void __launch_bounds__(256)
 gemm_generic_kernel(const TIn* __restrict__ x, const TIn* __restrict__ w, TOut* __restrict__ out,
-                    int M, int N, int K) {
+                    int M, int N, int K, int act) {
   __shared__ float xs[GG_BK][GG_BM + 4];
   __shared__ float ws[GG_BK][GG_BN + 4];
   pdl_launch_dependents();
@@ -60,26 +60,28 @@ gemm_generic_kernel(const TIn* __restrict__ x, const TIn* __restrict__ w, TOut* 
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int gn = n0 + tx * 4 + j;
-      if (gn < N) out[(size_t)gm * N + gn] = from_f32<TOut>(acc[i][j]);
+      if (gn < N) out[(size_t)gm * N + gn] = from_f32<TOut>(act_exact(acc[i][j], act));
     }
   }
 }
 
 extern "C" int qe_linear_generic(const void* x, const void* w, void* out, int M, int N, int K,
-                                 int dtype, int out_f32, cudaStream_t stream) {
+                                 int dtype, int out_mode, cudaStream_t stream) {
+  const int out_f32 = out_mode & 1, act = out_mode >> 1;       // (the activation of the sums: common.cuh)
+  if (act < 0 || act > QE_ACT_MAX) QE_REFUSE("linear: unknown activation %d", act);
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0) QE_REFUSE("linear: K must be positive");
   dim3 grid((N + GG_BN - 1) / GG_BN, (M + GG_BM - 1) / GG_BM);
   if (grid.y > 65535) QE_REFUSE("linear: M %d is too large for the generic kernel", M);
   if (dtype == QE_DTYPE_F32) {
-    qe_launch(gemm_generic_kernel<float, float>, grid, dim3(256), 0, stream, (const float*)x, (const float*)w, (float*)out, M, N, K);
+    qe_launch(gemm_generic_kernel<float, float>, grid, dim3(256), 0, stream, (const float*)x, (const float*)w, (float*)out, M, N, K, act);
   } else if (dtype == QE_DTYPE_BF16) {
     if (out_f32)
       qe_launch(gemm_generic_kernel<__nv_bfloat16, float>, grid, dim3(256), 0, stream,
-          (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (float*)out, M, N, K);
+          (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (float*)out, M, N, K, act);
     else
       qe_launch(gemm_generic_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(256), 0, stream,
-          (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, M, N, K);
+          (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, M, N, K, act);
   } else QE_REFUSE("linear: unknown dtype %d", dtype);
   QE_CHECK_LAUNCH("linear_generic");
   return 0;

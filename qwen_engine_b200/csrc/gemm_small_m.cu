@@ -248,8 +248,11 @@ static int dispatch_small_m(const void* x, const void* w, void* out, int M, int 
 
 // Returns 0 when run, 1 when refused (qe_last_error says why), 2 on a launch error.
 extern "C" int qe_linear_small_m(const void* x, const void* w, void* out, int M, int N, int K,
-                                 int out_f32, cudaStream_t stream) {
-  return dispatch_small_m<X_PLAIN, false>(x, w, out, M, N, K, out_f32, stream);
+                                 int out_mode, cudaStream_t stream) {
+  FuseArgs na{};
+  na.act = out_mode >> 1;                           // (the activation of the sums: common.cuh)
+  if (na.act < 0 || na.act > QE_ACT_MAX) QE_REFUSE("linear_small_m: unknown activation %d", na.act);
+  return dispatch_small_m<X_PLAIN, false>(x, w, out, M, N, K, out_mode & 1, stream, na);
 }
 
 // out[M, N] = (silu(gate_up[:, :K]) * gate_up[:, K:]) · w[N, K]^T: the activation of the feed-forward

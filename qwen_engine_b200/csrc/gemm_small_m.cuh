@@ -57,6 +57,7 @@ struct FuseArgs {
   // and a kernel that starts on weights that are already on the chip is done sooner.
   const unsigned char* next_w;
   unsigned long long next_bytes;
+  int act;                          // without RESID: the activation of the sums (common.cuh: act_for)
 };
 
 // a chunk of weights: 64 k of 16 rows = four 16-byte loads per lane (a: row g, b: row g + 8); where a CTA has 8
@@ -295,7 +296,7 @@ __device__ __forceinline__ void gsm_cta(const __nv_bfloat16* __restrict__ x, con
     };
     if (!RESID) {
       if (m >= M || n >= N) continue;
-      out[(size_t)m * N + n] = from_f32<TOut>(total());
+      out[(size_t)m * N + n] = from_f32<TOut>(act_for<TOut>(total(), na.act));
     } else {
       // whole warps run this loop (ROWS MW is a multiple of 32); lanes outside the matrix add zero
       float v = 0.f;

@@ -44,7 +44,7 @@ struct __align__(1024) TcSmem {
 template <typename TOut, int BN, int STAGES, bool STARVED = false>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                    TOut* __restrict__ out, int M, int N, int K, int starved_limit) {
+                    TOut* __restrict__ out, int M, int N, int K, int starved_limit, int act) {
   extern __shared__ unsigned char smem_raw[];
   using Smem = TcSmem<BN, STAGES>;
   constexpr uint32_t TMEM_COLS = 2 * BN;
@@ -168,6 +168,10 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           __syncwarp();
           if (lane == 0) mbar_arrive(&sm.acc_empty[buf]);
         }
+        if (act) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(act_for<TOut>(__uint_as_float(r[j]), act));
+        }
         if (row < M && n0 + c0 < N) {
           TOut* dst = out + (size_t)row * N + n0 + c0;
           if (n0 + c0 + 32 <= N && (N % 8) == 0) {
@@ -229,7 +233,7 @@ extern "C" void qe_gemm_tc_clear_status() {
 }
 
 template <int BN, int STAGES>
-static int launch_tc(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, int sms, cudaStream_t stream) {
+static int launch_tc(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, int sms, cudaStream_t stream, int act) {
   CUtensorMap map_x, map_w;
   if (!get_map(x, M, K, TC_BM, &map_x) || !get_map(w, N, K, BN, &map_w)) return 1;
   const size_t smem = sizeof(TcSmem<BN, STAGES>) + 1024;
@@ -243,9 +247,9 @@ static int launch_tc(const void* x, const void* w, void* out, int M, int N, int 
   const long tiles = (long)((N + BN - 1) / BN) * ((M + TC_BM - 1) / TC_BM);
   const dim3 grid((unsigned)(tiles < sms ? tiles : sms));
   if (out_f32)
-    qe_launch(gemm_tcgen05_kernel<float, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (float*)out, M, N, K, 0);
+    qe_launch(gemm_tcgen05_kernel<float, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (float*)out, M, N, K, 0, act);
   else
-    qe_launch(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (__nv_bfloat16*)out, M, N, K, 0);
+    qe_launch(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (__nv_bfloat16*)out, M, N, K, 0, act);
   QE_CHECK_LAUNCH("linear_tcgen05");
   return 0;
 }
@@ -265,7 +269,7 @@ extern "C" int qe_gemm_tc_selftest_starved(const void* x, const void* w, void* o
   cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<__nv_bfloat16, 128, 6, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) QE_REFUSE("selftest: shared memory %zu: %s", smem, cudaGetErrorString(e));
   qe_launch(gemm_tcgen05_kernel<__nv_bfloat16, 128, 6, true>, dim3(1), dim3(TC_THREADS), smem, stream, map_x, map_w,
-            (__nv_bfloat16*)out, M, N, K, limit);
+            (__nv_bfloat16*)out, M, N, K, limit, 0);
   QE_CHECK_LAUNCH("selftest");
   return 0;
 }
@@ -282,14 +286,16 @@ static int sm_count() {
   return sms[dev];
 }
 
-extern "C" int qe_linear_tcgen05(const void* x, const void* w, void* out, int M, int N, int K, int out_f32,
+extern "C" int qe_linear_tcgen05(const void* x, const void* w, void* out, int M, int N, int K, int out_mode,
                                  cudaStream_t stream) {
+  const int out_f32 = out_mode & 1, act = out_mode >> 1;       // (the activation of the sums: common.cuh)
+  if (act < 0 || act > QE_ACT_MAX) QE_REFUSE("linear_tcgen05: unknown activation %d", act);
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) QE_REFUSE("linear_tcgen05: K = %d is not a positive multiple of 8", K);
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) QE_REFUSE("linear_tcgen05: operands must be 16-byte aligned");
   const int sms = sm_count();
   // wide tiles reuse the fetched rows of x twice as often; narrow ones when wide ones would leave SMs idle
   const long wide_tiles = (long)((N + 255) / 256) * ((M + TC_BM - 1) / TC_BM);
-  if (wide_tiles >= sms) return launch_tc<256, 4>(x, w, out, M, N, K, out_f32, sms, stream);
-  return launch_tc<128, 6>(x, w, out, M, N, K, out_f32, sms, stream);
+  if (wide_tiles >= sms) return launch_tc<256, 4>(x, w, out, M, N, K, out_f32, sms, stream, act);
+  return launch_tc<128, 6>(x, w, out, M, N, K, out_f32, sms, stream, act);
 }

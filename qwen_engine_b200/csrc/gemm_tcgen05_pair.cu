@@ -111,7 +111,7 @@ __device__ __forceinline__ void pr_store_block(unsigned char* wst, const uint32_
 // in flight before the first is used (a load from another CTA's shared memory takes some hundreds of cycles).
 template <typename TOut, int BN, int S>
 __device__ __forceinline__ void pr_meet_shares(const unsigned char* stg, TOut* __restrict__ out, int M, int N, int m0, int n0,
-                                               uint32_t rank, uint32_t cpair) {
+                                               uint32_t rank, uint32_t cpair, int act) {
   constexpr int CPR = (BN / 4) / S;                  // 16-byte chunks of a row that this CTA finishes
   constexpr int BATCH = 4;
   static_assert((PR_BM * CPR) % (PR_EPI_WARPS * 32 * BATCH) == 0, "whole batches per thread");
@@ -137,6 +137,10 @@ __device__ __forceinline__ void pr_meet_shares(const unsigned char* stg, TOut* _
       float4 acc = v[b][0];                          // in the order of the shares
 #pragma unroll
       for (int sp = 1; sp < S; ++sp) { acc.x += v[b][sp].x; acc.y += v[b][sp].y; acc.z += v[b][sp].z; acc.w += v[b][sp].w; }
+      if (act) {
+        acc.x = act_for<TOut>(acc.x, act); acc.y = act_for<TOut>(acc.y, act);
+        acc.z = act_for<TOut>(acc.z, act); acc.w = act_for<TOut>(acc.w, act);
+      }
       const int row = m0 + rr, col = n0 + chunk * 4;
       if (row < M && col < N) {                      // N is a multiple of 8 here (the launcher's rule)
         if constexpr (sizeof(TOut) == 2) {
@@ -498,6 +502,12 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive_cluster(smem_u32(&sm.acc_empty[buf]) & TC_PEER_BIT_MASK);
+        if (gate_act) {                              // (a plain product: the activation of its sums)
+#pragma unroll
+          for (int q = 0; q < NLD; ++q)
+#pragma unroll
+            for (int j = 0; j < 32; ++j) r[q][j] = __float_as_uint(act_fast(__uint_as_float(r[q][j]), gate_act));
+        }
         const int r_first = m0 + quarter * 32;
 #pragma unroll
         for (int h = 0; h < NLD / 2; ++h) {
@@ -525,6 +535,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
           tc_fence_before();
           __syncwarp();
           if (lane == 0) mbar_arrive_cluster(smem_u32(&sm.acc_empty[buf]) & TC_PEER_BIT_MASK);
+        }
+        if (gate_act) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(act_for<TOut>(__uint_as_float(r[j]), gate_act));
         }
         if (row < M && n0 + c0 < N) {
           TOut* dst = out + (size_t)row * N + n0 + c0;
@@ -556,8 +570,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
     if (warp >= 2 && split_staged) {
       const int tile = pair;
       const int m0 = (tile / n_blocks) * 2 * PR_BM + (int)rank * PR_BM, n0 = (tile % n_blocks) * BN;
-      if (splits == 2) pr_meet_shares<TOut, BN, 2>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair);
-      else pr_meet_shares<TOut, BN, 4>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair);
+      if (splits == 2) pr_meet_shares<TOut, BN, 2>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
+      else pr_meet_shares<TOut, BN, 4>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
     }
   }
   // both CTAs meet here: neither leaves while the other may still signal its barriers, read its
@@ -707,8 +721,10 @@ extern "C" void qe_gemm_tc_pair_clear_status() {
 }
 
 // Returns 0 when run, 1 when refused (qe_last_error says why), 2 on a launch error.
-extern "C" int qe_linear_tcgen05_pair(const void* x, const void* w, void* out, int M, int N, int K, int out_f32,
+extern "C" int qe_linear_tcgen05_pair(const void* x, const void* w, void* out, int M, int N, int K, int out_mode,
                                       cudaStream_t stream) {
+  const int out_f32 = out_mode & 1, act = out_mode >> 1;       // (the activation of the sums: common.cuh)
+  if (act < 0 || act > QE_ACT_MAX) QE_REFUSE("linear_tcgen05_pair: unknown activation %d", act);
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || K % 8) QE_REFUSE("linear_tcgen05_pair: K = %d is not a positive multiple of 8", K);
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) QE_REFUSE("linear_tcgen05_pair: operands must be 16-byte aligned");
@@ -717,9 +733,9 @@ extern "C" int qe_linear_tcgen05_pair(const void* x, const void* w, void* out, i
   if (sms < 2) QE_REFUSE("linear_tcgen05_pair: needs at least two SMs");
   // wide tiles, wide tiles with K split over 2 or 4 pairs, or narrow tiles: see qe_tc_product_plan
   const int plan = qe_tc_product_plan(M, N, K, 1);
-  if (plan == 2) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream);
-  if (plan >= 3) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, plan == 3 ? 2 : 4);
-  return launch_pair<128, 8>(x, w, out, M, N, K, out_f32, sms, stream);
+  if (plan == 2) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, 1, act);
+  if (plan >= 3) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, plan == 3 ? 2 : 4, act);
+  return launch_pair<128, 8>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, 1, act);
 }
 
 // out[M, I] = silu(x · w[:I]^T) * (x · w[I:]^T) for the stacked gate and up weights w [2 I, K] (see SWIGLU

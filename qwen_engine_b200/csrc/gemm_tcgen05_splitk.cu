@@ -44,7 +44,7 @@ struct __align__(1024) SkSmem {
 template <typename TOut, int S, int STAGES, bool RESID>
 __global__ void __launch_bounds__(SK_THREADS, 1)
 gemm_tcgen05_splitk_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-                           TOut* __restrict__ out, int M, int N, int K) {
+                           TOut* __restrict__ out, int M, int N, int K, int act) {
   extern __shared__ unsigned char smem_raw[];
   using Smem = SkSmem<STAGES>;
   constexpr uint32_t TMEM_COLS = SK_BT;
@@ -162,6 +162,10 @@ gemm_tcgen05_splitk_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
       float4 acc = v[0];
 #pragma unroll
       for (int s = 1; s < S; ++s) { acc.x += v[s].x; acc.y += v[s].y; acc.z += v[s].z; acc.w += v[s].w; }
+      if (!RESID && act) {
+        acc.x = act_for<TOut>(acc.x, act); acc.y = act_for<TOut>(acc.y, act);
+        acc.z = act_for<TOut>(acc.z, act); acc.w = act_for<TOut>(acc.w, act);
+      }
       if (n < N) {                                    // N % 4 == 0: the four lie inside together
         TOut* dst = out + (size_t)c * N + n;
         if constexpr (sizeof(TOut) == 4) {
@@ -192,7 +196,7 @@ gemm_tcgen05_splitk_kernel(const __grid_constant__ CUtensorMap map_w, const __gr
 }
 
 template <typename TOut, int S, int STAGES, bool RESID>
-static int launch_splitk_as(const CUtensorMap& map_w, const CUtensorMap& map_x, void* out, int M, int N, int K, cudaStream_t stream) {
+static int launch_splitk_as(const CUtensorMap& map_w, const CUtensorMap& map_x, void* out, int M, int N, int K, cudaStream_t stream, int act) {
   const size_t smem = sizeof(SkSmem<STAGES>) + 1024;
   static bool configured = false;
   if (!configured) {
@@ -203,13 +207,13 @@ static int launch_splitk_as(const CUtensorMap& map_w, const CUtensorMap& map_x, 
   }
   const dim3 grid((unsigned)((N + SK_BM - 1) / SK_BM) * S);
   qe_launch_cluster(gemm_tcgen05_splitk_kernel<TOut, S, STAGES, RESID>, grid, dim3(SK_THREADS), smem, stream, (unsigned)S,
-                    map_w, map_x, (TOut*)out, M, N, K);
+                    map_w, map_x, (TOut*)out, M, N, K, act);
   QE_CHECK_LAUNCH("linear_tcgen05_splitk");
   return 0;
 }
 
 template <int S>
-static int launch_splitk(const void* x, const void* w, void* out, int M, int N, int K, int mode, cudaStream_t stream) {
+static int launch_splitk(const void* x, const void* w, void* out, int M, int N, int K, int mode, cudaStream_t stream, int act) {
   CUtensorMap map_w, map_x;
   {
     const uint64_t dims[2] = {(uint64_t)K, (uint64_t)N};
@@ -223,9 +227,9 @@ static int launch_splitk(const void* x, const void* w, void* out, int M, int N, 
     const uint32_t box[2] = {SK_BK, SK_BT};
     if (!qe_tensor_map_bf16(x, 2, dims, strides, box, &map_x)) return 1;
   }
-  if (mode == 2) return launch_splitk_as<float, S, 6, true>(map_w, map_x, out, M, N, K, stream);
-  if (mode == 1) return launch_splitk_as<float, S, 6, false>(map_w, map_x, out, M, N, K, stream);
-  return launch_splitk_as<__nv_bfloat16, S, 6, false>(map_w, map_x, out, M, N, K, stream);
+  if (mode == 2) return launch_splitk_as<float, S, 6, true>(map_w, map_x, out, M, N, K, stream, act);
+  if (mode == 1) return launch_splitk_as<float, S, 6, false>(map_w, map_x, out, M, N, K, stream, act);
+  return launch_splitk_as<__nv_bfloat16, S, 6, false>(map_w, map_x, out, M, N, K, stream, act);
 }
 
 extern "C" int qe_gemm_tc_splitk_status() {
@@ -243,14 +247,17 @@ extern "C" void qe_gemm_tc_splitk_clear_status() {
 // product.  Returns 0 when run, 1 when refused (qe_last_error says why), 2 on a launch error.
 extern "C" int qe_linear_tcgen05_splitk(const void* x, const void* w, void* out, int M, int N, int K, int splits, int mode,
                                         cudaStream_t stream) {
+  const int act = mode >> 2;                          // (modes 0 and 1: the activation of the sums, common.cuh)
+  mode &= 3;
+  if (act < 0 || act > QE_ACT_MAX || (act && mode == 2)) QE_REFUSE("linear_tcgen05_splitk: activation %d", act);
   if (M <= 0 || N <= 0) return 0;
   if (M > SK_BT) QE_REFUSE("linear_tcgen05_splitk: M = %d is above %d", M, SK_BT);
   if (K <= 0 || K % 8) QE_REFUSE("linear_tcgen05_splitk: K = %d is not a positive multiple of 8", K);
   if (N % 4) QE_REFUSE("linear_tcgen05_splitk: N = %d is not a multiple of 4", N);
   if (mode < 0 || mode > 2) QE_REFUSE("linear_tcgen05_splitk: mode %d", mode);
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) QE_REFUSE("linear_tcgen05_splitk: operands must be 16-byte aligned");
-  if (splits == 2) return launch_splitk<2>(x, w, out, M, N, K, mode, stream);
-  if (splits == 4) return launch_splitk<4>(x, w, out, M, N, K, mode, stream);
-  if (splits == 8) return launch_splitk<8>(x, w, out, M, N, K, mode, stream);
+  if (splits == 2) return launch_splitk<2>(x, w, out, M, N, K, mode, stream, act);
+  if (splits == 4) return launch_splitk<4>(x, w, out, M, N, K, mode, stream, act);
+  if (splits == 8) return launch_splitk<8>(x, w, out, M, N, K, mode, stream, act);
   QE_REFUSE("linear_tcgen05_splitk: %d splits (2, 4 or 8)", splits);
 }

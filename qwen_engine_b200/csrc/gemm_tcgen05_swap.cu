@@ -34,7 +34,7 @@ struct __align__(1024) SwSmem {
 template <typename TOut, int BT, int STAGES>
 __global__ void __launch_bounds__(SW_THREADS, 1)
 gemm_tcgen05_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x,
-                         TOut* __restrict__ out, int M, int N, int K) {
+                         TOut* __restrict__ out, int M, int N, int K, int act) {
   extern __shared__ unsigned char smem_raw[];
   using Smem = SwSmem<BT, STAGES>;
   constexpr uint32_t TMEM_COLS = BT < 32 ? 32 : BT;
@@ -122,7 +122,7 @@ gemm_tcgen05_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid
         if (n < N) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
-            if (c0 + j < M) out[(size_t)(c0 + j) * N + n] = from_f32<TOut>(__uint_as_float(r[j]));
+            if (c0 + j < M) out[(size_t)(c0 + j) * N + n] = from_f32<TOut>(act_for<TOut>(__uint_as_float(r[j]), act));
         }
       }
     }
@@ -139,7 +139,7 @@ gemm_tcgen05_swap_kernel(const __grid_constant__ CUtensorMap map_w, const __grid
 }
 
 template <int BT, int STAGES>
-static int launch_swap(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, cudaStream_t stream) {
+static int launch_swap(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, cudaStream_t stream, int act) {
   CUtensorMap map_w, map_x;
   {
     const uint64_t dims[2] = {(uint64_t)K, (uint64_t)N};
@@ -163,9 +163,9 @@ static int launch_swap(const void* x, const void* w, void* out, int M, int N, in
   }
   const dim3 grid((unsigned)((N + SW_BM - 1) / SW_BM));
   if (out_f32)
-    qe_launch(gemm_tcgen05_swap_kernel<float, BT, STAGES>, grid, dim3(SW_THREADS), smem, stream, map_w, map_x, (float*)out, M, N, K);
+    qe_launch(gemm_tcgen05_swap_kernel<float, BT, STAGES>, grid, dim3(SW_THREADS), smem, stream, map_w, map_x, (float*)out, M, N, K, act);
   else
-    qe_launch(gemm_tcgen05_swap_kernel<__nv_bfloat16, BT, STAGES>, grid, dim3(SW_THREADS), smem, stream, map_w, map_x, (__nv_bfloat16*)out, M, N, K);
+    qe_launch(gemm_tcgen05_swap_kernel<__nv_bfloat16, BT, STAGES>, grid, dim3(SW_THREADS), smem, stream, map_w, map_x, (__nv_bfloat16*)out, M, N, K, act);
   QE_CHECK_LAUNCH("linear_tcgen05_swap");
   return 0;
 }
@@ -181,13 +181,15 @@ extern "C" void qe_gemm_tc_swap_clear_status() {
 }
 
 // 1 <= M <= 256.  Returns 0 when run, 1 when refused (qe_last_error says why), 2 on a launch error.
-extern "C" int qe_linear_tcgen05_swap(const void* x, const void* w, void* out, int M, int N, int K, int out_f32,
+extern "C" int qe_linear_tcgen05_swap(const void* x, const void* w, void* out, int M, int N, int K, int out_mode,
                                       cudaStream_t stream) {
+  const int out_f32 = out_mode & 1, act = out_mode >> 1;       // (the activation of the sums: common.cuh)
+  if (act < 0 || act > QE_ACT_MAX) QE_REFUSE("linear_tcgen05_swap: unknown activation %d", act);
   if (M <= 0 || N <= 0) return 0;
   if (M > 256) QE_REFUSE("linear_tcgen05_swap: M = %d is above 256", M);
   if (K <= 0 || K % 8) QE_REFUSE("linear_tcgen05_swap: K = %d is not a positive multiple of 8", K);
   if (((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) & 15) QE_REFUSE("linear_tcgen05_swap: operands must be 16-byte aligned");
-  if (M <= 64) return launch_swap<64, 8>(x, w, out, M, N, K, out_f32, stream);
-  if (M <= 128) return launch_swap<128, 6>(x, w, out, M, N, K, out_f32, stream);
-  return launch_swap<256, 4>(x, w, out, M, N, K, out_f32, stream);
+  if (M <= 64) return launch_swap<64, 8>(x, w, out, M, N, K, out_f32, stream, act);
+  if (M <= 128) return launch_swap<128, 6>(x, w, out, M, N, K, out_f32, stream, act);
+  return launch_swap<256, 4>(x, w, out, M, N, K, out_f32, stream, act);
 }

@@ -10,7 +10,10 @@
 //
 //   qe_latent_prepare   per token: RMS norm of the latent and rotation of the shared key part, both written to the
 //                       token's cache slot; rotation of every head's rotated query part into the packed query
-//   qe_head_linear      out[t, h, :N] = W[h] x[t, h, :K], one matrix per head (the two folds above)
+//   qe_head_linear      out[t, h, :N] = W[h] x[t, h, :K], one matrix per head (the two folds above), optionally times
+//                       sigmoid(gate[t, h]) (a mixer that gates every head by one number)
+//
+// A layer that reads another layer's cache (write_kv 0) has no latent of its own: only the queries' parts are rotated.
 //
 // Norm, angles and rotation in float32; one rounding into the cache and into the packed query.
 #include "tile_product.cuh"
@@ -89,11 +92,13 @@ extern "C" int qe_latent_prepare(const void* down, long ld_down, const void* q, 
   return 0;
 }
 
+__device__ __forceinline__ float hl_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
 // out[t * ldo + h * ldo_h + n] = sum_k w[h][n][k] * x[t * ldx + h * ldx_h + k]
 template <typename T>
 __global__ void __launch_bounds__(TP_THREADS)
 head_linear_kernel(const T* __restrict__ x, long ldx, long ldx_h, const T* __restrict__ w, T* __restrict__ out, long ldo,
-                   long ldo_h, int M, int N, int K) {
+                   long ldo_h, int M, int N, int K, const T* __restrict__ gate, long ldg) {
   __shared__ TpSmem<T, 1> sm;
   TpAcc<T, 1> acc;
   const int m0 = blockIdx.x * TP_BM, n0 = blockIdx.y * TP_BN, h = blockIdx.z;
@@ -104,13 +109,14 @@ head_linear_kernel(const T* __restrict__ x, long ldx, long ldx_h, const T* __res
       [&](int r) -> const T* { return m0 + r < M ? x + (size_t)(m0 + r) * ldx + (size_t)h * ldx_h : nullptr; },
       [&](int, int n) -> const T* { return n0 + n < N ? wh + (size_t)(n0 + n) * K : nullptr; });
   tile_for_each<T, 1>(acc, [&](int r, int n, float v, float) {
-    if (m0 + r < M && n0 + n < N) out[(size_t)(m0 + r) * ldo + (size_t)h * ldo_h + n0 + n] = from_f32<T>(v);
+    if (m0 + r < M && n0 + n < N) out[(size_t)(m0 + r) * ldo + (size_t)h * ldo_h + n0 + n] = from_f32<T>(gate ? v * hl_sigmoid(to_f32(gate[(size_t)(m0 + r) * ldg + h])) : v);
   });
 }
 
 __global__ void __launch_bounds__(FP_THREADS)
 head_linear_fast_kernel(const __nv_bfloat16* __restrict__ x, long ldx, long ldx_h, const __nv_bfloat16* __restrict__ w,
-                        __nv_bfloat16* __restrict__ out, long ldo, long ldo_h, int M, int N, int K) {
+                        __nv_bfloat16* __restrict__ out, long ldo, long ldo_h, int M, int N, int K,
+                        const __nv_bfloat16* __restrict__ gate, long ldg) {
   extern __shared__ __align__(16) unsigned char fp_smem[];
   FpAcc acc;
   constexpr int BN = FpShape<1>::BN;
@@ -122,12 +128,12 @@ head_linear_fast_kernel(const __nv_bfloat16* __restrict__ x, long ldx, long ldx_
       [&](int r) -> const __nv_bfloat16* { return m0 + r < M ? x + (size_t)(m0 + r) * ldx + (size_t)h * ldx_h : nullptr; },
       [&](int, int n) -> const __nv_bfloat16* { return n0 + n < N ? wh + (size_t)(n0 + n) * K : nullptr; });
   fast_tile_for_each<1>(acc, [&](int r, int n, float v, float) {
-    if (m0 + r < M && n0 + n < N) out[(size_t)(m0 + r) * ldo + (size_t)h * ldo_h + n0 + n] = __float2bfloat16_rn(v);
+    if (m0 + r < M && n0 + n < N) out[(size_t)(m0 + r) * ldo + (size_t)h * ldo_h + n0 + n] = __float2bfloat16_rn(gate ? v * hl_sigmoid(to_f32(gate[(size_t)(m0 + r) * ldg + h])) : v);
   });
 }
 
 extern "C" int qe_head_linear(const void* x, long ldx, long ldx_h, const void* w, void* out, long ldo, long ldo_h,
-                              int M, int H, int N, int K, int dtype, cudaStream_t stream) {
+                              int M, int H, int N, int K, int dtype, const void* gate, long ldg, cudaStream_t stream) {
   if (M <= 0 || H <= 0 || N <= 0) return 0;
   if (K < 1 || H > 65535) QE_REFUSE("head_linear: K = %d, %d heads", K, H);
   if (dtype == QE_DTYPE_BF16 && K % 8 == 0 && ldx % 8 == 0 && ldx_h % 8 == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0) {
@@ -141,14 +147,15 @@ extern "C" int qe_head_linear(const void* x, long ldx, long ldx_h, const void* w
     dim3 fgrid((M + FP_BM - 1) / FP_BM, (N + FpShape<1>::BN - 1) / FpShape<1>::BN, H);
     if (fgrid.y > 65535) QE_REFUSE("head_linear: N = %d is too wide", N);
     qe_launch(head_linear_fast_kernel, fgrid, dim3(FP_THREADS), FP_SMEM_BYTES, stream, (const __nv_bfloat16*)x, ldx, ldx_h,
-              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ldo_h, M, N, K);
+              (const __nv_bfloat16*)w, (__nv_bfloat16*)out, ldo, ldo_h, M, N, K,
+              (const __nv_bfloat16*)gate, ldg);
     QE_CHECK_LAUNCH("head_linear");
     return 0;
   }
   dim3 grid((M + TP_BM - 1) / TP_BM, (N + TP_BN - 1) / TP_BN, H);
   if (grid.y > 65535) QE_REFUSE("head_linear: N = %d is too wide", N);
 #define HL(TT) qe_launch(head_linear_kernel<TT>, grid, dim3(TP_THREADS), 0, stream, (const TT*)x, ldx, ldx_h, (const TT*)w, \
-                         (TT*)out, ldo, ldo_h, M, N, K)
+                         (TT*)out, ldo, ldo_h, M, N, K, (const TT*)gate, ldg)
   if (dtype == QE_DTYPE_F32) HL(float);
   else if (dtype == QE_DTYPE_BF16) HL(__nv_bfloat16);
   else QE_REFUSE("head_linear: unknown dtype %d", dtype);

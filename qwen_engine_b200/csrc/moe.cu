@@ -3,11 +3,16 @@
 //
 //   qe_moe_route       z = W_r h + b in float32 per token; the `top` largest (the lower index wins a tie); weights =
 //                      softmax over the chosen logits alone.  Second scoring: s = softmax(z) over all outputs, the `top`
-//                      largest of s + correction are chosen, the weights are their s as it is
+//                      largest of s + correction are chosen, the weights are their s as it is.  Third: every output is
+//                      scored alone by a sigmoid, the weights are the chosen scores as they are.  Fourth: the same scores,
+//                      divided by their sum (+ 1e-20) and times a constant.  Behind the chosen experts a token may name
+//                      `n_always` more that every token uses (a shared expert, cut into pieces of the experts' size): their
+//                      weight is sigmoid(z[E]), the router's matrix then has one row more
 //   qe_moe_sort        the (token, choice) pairs ordered by expert: offsets[E + 1], the pairs of every expert side by
 //                      side, and where each pair went.  One CTA.  Which pair of an expert comes first is not fixed
 //                      (atomics); nothing depends on it, since every pair's row is computed alone
 //   qe_moe_gate_up     act[p, :] = glu(W_gate_e x_t, W_up_e x_t) for the pair p = (t, e) in sorted order
+//   qe_moe_up          act[p, :] = f(W_up_e x_t) for experts without a gate
 //   qe_moe_down        y[p, :] = W_down_e act[p, :], float32
 //   qe_moe_combine     out[t, :] = sum over the token's choices, in their order, of weight x y[place of the pair]; a choice
 //                      at or beyond the experts that have weights stands for an expert that hands its input on: x[t, :]
@@ -24,8 +29,8 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                  int* __restrict__ top_idx, float* __restrict__ top_w, int T_tokens, int W, int E, int top, int scoring,
-                 const float* __restrict__ correction) {
-  extern __shared__ float route_smem[];             // the token's row [W], then its logits [E]
+                 const float* __restrict__ correction, float weight_scale, int n_always) {
+  extern __shared__ float route_smem[];             // the token's row [W], then its logits [E (+ 1)]
   float* xs = route_smem;
   float* z = route_smem + ((W + 3) & ~3);
   pdl_launch_dependents();
@@ -37,7 +42,8 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
   __syncthreads();
   // a warp per expert in turn; a lane's share of the row in four sums that do not wait for each other, then the lanes' sums
   // in a fixed order: a logit's bits depend on W alone
-  for (int e = warp; e < E; e += warps) {
+  const int n_out = E + (n_always > 0 ? 1 : 0);
+  for (int e = warp; e < n_out; e += warps) {
     const float* wr = w + (size_t)e * W;
     float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
     int d = lane;
@@ -65,10 +71,15 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
   }
   __syncthreads();
   if (warp != 0) return;
+  const size_t first = (size_t)t * (top + n_always);
+  for (int j = lane; j < n_always; j += 32) {
+    top_idx[first + top + j] = E + j;
+    top_w[first + top + j] = 1.f / (1.f + expf(-z[E]));
+  }
   if (scoring == 1) {
     // scores over all outputs: the largest logit and the sum of the exponentials lane by lane, then over the lanes in a
     // fixed order; the choice looks at score + correction, the weight is the score
-    float* sc = z + E;                               // the scores, behind the logits (which become the choice values)
+    float* sc = z + E + 1;                           // the scores, behind the logits (which become the choice values)
     float m = -INFINITY;
     for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
 #pragma unroll
@@ -90,7 +101,7 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
         if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
       }
       if (at == 0x7fffffff) at = 0;
-      if (lane == 0) { top_idx[(size_t)t * top + j] = at; top_w[(size_t)t * top + j] = sc[at]; z[at] = -INFINITY; }
+      if (lane == 0) { top_idx[first + j] = at; top_w[first + j] = sc[at]; z[at] = -INFINITY; }
       __syncwarp();
     }
     return;
@@ -110,25 +121,35 @@ moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const flo
     if (at == 0x7fffffff) at = 0;                  // (only logits that are not numbers: the row is lost anyway)
     chosen[j] = best;
     if (j == 0) zmax = best;
-    if (lane == 0) { top_idx[(size_t)t * top + j] = at; z[at] = -INFINITY; }
+    if (lane == 0) { top_idx[first + j] = at; z[at] = -INFINITY; }
     __syncwarp();
   }
   if (scoring == 2) {
     // every expert scored alone: sigmoid(z); the largest logits are the largest scores; the weights are the scores as they are
-    if (lane == 0) for (int j = 0; j < top; ++j) top_w[(size_t)t * top + j] = 1.f / (1.f + expf(-chosen[j]));
+    if (lane == 0) for (int j = 0; j < top; ++j) top_w[first + j] = 1.f / (1.f + expf(-chosen[j]));
+    return;
+  }
+  if (scoring == 3) {
+    // the same scores, made to sum to one and scaled
+    float s = 0.f;
+    for (int j = 0; j < top; ++j) { chosen[j] = 1.f / (1.f + expf(-chosen[j])); s += chosen[j]; }
+    const float norm = 1.f / (s + 1e-20f);
+    if (lane == 0) for (int j = 0; j < top; ++j) top_w[first + j] = chosen[j] * norm * weight_scale;
     return;
   }
   float sum = 0.f;
   for (int j = 0; j < top; ++j) { chosen[j] = expf(chosen[j] - zmax); sum += chosen[j]; }
-  if (lane == 0) for (int j = 0; j < top; ++j) top_w[(size_t)t * top + j] = chosen[j] / sum;
+  if (lane == 0) for (int j = 0; j < top; ++j) top_w[first + j] = chosen[j] / sum;
 }
 
 extern "C" int qe_moe_route(const void* x, const float* w, const float* bias, int* top_idx, float* top_w, int T, int W,
-                            int E, int top, int dtype, int scoring, const float* correction, cudaStream_t stream) {
+                            int E, int top, int dtype, int scoring, const float* correction, float weight_scale, int n_always,
+                            cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (n_always < 0 || n_always + E > MOE_MAX_E) QE_REFUSE("moe_route: %d experts beside %d", n_always, E);
   if (E < 1 || E > MOE_MAX_E || top < 1 || top > MOE_MAX_TOP || top > E) QE_REFUSE("moe_route: %d of %d experts", top, E);
-  if (scoring < 0 || scoring > 2) QE_REFUSE("moe_route: unknown scoring %d", scoring);
-  const size_t smem = ((size_t)((W + 3) & ~3) + 2 * (size_t)E) * sizeof(float);
+  if (scoring < 0 || scoring > 3) QE_REFUSE("moe_route: unknown scoring %d", scoring);
+  const size_t smem = ((size_t)((W + 3) & ~3) + 2 * (size_t)E + 1) * sizeof(float);
   if (smem > 160 * 1024) QE_REFUSE("moe_route: a row of %d channels does not fit shared memory", W);
   static bool configured = false;
   if (!configured) {
@@ -137,7 +158,7 @@ extern "C" int qe_moe_route(const void* x, const float* w, const float* bias, in
     if (e != cudaSuccess) QE_REFUSE("moe_route: shared memory: %s", cudaGetErrorString(e));
     configured = true;
   }
-#define MR(TT) qe_launch(moe_route_kernel<TT>, dim3(T), dim3(128), smem, stream, (const TT*)x, w, bias, top_idx, top_w, T, W, E, top, scoring, correction)
+#define MR(TT) qe_launch(moe_route_kernel<TT>, dim3(T), dim3(128), smem, stream, (const TT*)x, w, bias, top_idx, top_w, T, W, E, top, scoring, correction, weight_scale, n_always)
   if (dtype == QE_DTYPE_F32) MR(float);
   else if (dtype == QE_DTYPE_BF16) MR(__nv_bfloat16);
   else QE_REFUSE("moe_route: unknown dtype %d", dtype);
@@ -207,13 +228,16 @@ __device__ __forceinline__ float moe_glu(float v0, float v1, int act) {
   return g / (1.f + expf(-g)) * u;
 }
 
-// GLU = true: w [E, 2 I, K] (gate rows, then up rows), rows gathered from x by pair / top, out [P, I] in the compute type
-// GLU = false: w [E, N, K], rows are x[p], out float32 [P, N]
-template <typename T, bool GLU>
+// MOE_GLU: w [E, 2 I, K] (gate rows, then up rows), rows gathered from x by pair / top, out [P, I] in the compute type
+// MOE_ACT: w [E, I, K], rows gathered likewise, out [P, I] = f(product) in the compute type (f: common.cuh, act_for)
+// MOE_DOWN: w [E, N, K], rows are x[p], out float32 [P, N]
+enum { MOE_DOWN = 0, MOE_GLU = 1, MOE_ACT = 2 };
+template <typename T, int MODE>
 __global__ void __launch_bounds__(TP_THREADS)
 moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* __restrict__ offsets,
                    const int* __restrict__ sorted_pair, void* __restrict__ out_, int E, int N, int K, int top, int act,
                    const float* __restrict__ pair_w) {
+  constexpr bool GLU = MODE == MOE_GLU, GATHER = MODE != MOE_DOWN;
   __shared__ TpSmem<T, GLU ? 2 : 1> sm;
   __shared__ int s_tile[4];
   TpAcc<T, GLU ? 2 : 1> acc;
@@ -232,7 +256,7 @@ moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* 
   tile_product<T, GLU ? 2 : 1>(sm, acc, K,
       [&](int r) -> const T* {
         if (r >= rows) return nullptr;
-        return GLU ? x + (size_t)(sorted_pair[first + r] / top) * K : x + (size_t)(first + r) * K;
+        return GATHER ? x + (size_t)(sorted_pair[first + r] / top) * K : x + (size_t)(first + r) * K;
       },
       [&](int m, int n) -> const T* { return n0 + n < N ? we + ((size_t)m * N + n0 + n) * K : nullptr; });
   tile_for_each<T, GLU ? 2 : 1>(acc, [&](int r, int n, float v0, float v1) {
@@ -243,6 +267,9 @@ moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* 
       const float pw = pair_w ? pair_w[sorted_pair[first + r]] : 1.f;
       const float y = moe_glu<T>(v0 * pw, v1 * pw, act);
       ((T*)out_)[at] = from_f32<T>(y);
+    } else if constexpr (MODE == MOE_ACT) {
+      const float pw = pair_w ? pair_w[sorted_pair[first + r]] : 1.f;
+      ((T*)out_)[at] = from_f32<T>(act_exact(v0 * pw, act));
     } else {
       ((float*)out_)[at] = v0;
     }
@@ -250,9 +277,9 @@ moe_product_kernel(const T* __restrict__ x, const T* __restrict__ w, const int* 
 }
 
 // The same two products for bfloat16 rows on 16-byte boundaries, on the pipelined tile of 128 rows (tile_product.cuh).
-// K may be cut into gridDim.z shares of k_share channels (GLU = false only): share z adds up its channels alone and writes
+// K may be cut into gridDim.z shares of k_share channels (MOE_DOWN only): share z adds up its channels alone and writes
 // its sums to out + z * P * N; the combining kernel adds the shares in their order.
-template <bool GLU>
+template <int MODE>
 __global__ void __launch_bounds__(FP_THREADS)
 moe_product_fast_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, const int* __restrict__ offsets,
                         const int* __restrict__ sorted_pair, void* __restrict__ out_, int E, int N, int K, int top, int act,
@@ -260,6 +287,7 @@ moe_product_fast_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16
   extern __shared__ __align__(16) unsigned char fp_smem[];
   __shared__ int s_tile[4];
   FpAcc acc;
+  constexpr bool GLU = MODE == MOE_GLU, GATHER = MODE != MOE_DOWN;
   constexpr int NB = GLU ? 2 : 1;
   constexpr int BN = FpShape<NB>::BN;
   pdl_launch_dependents();
@@ -279,7 +307,7 @@ moe_product_fast_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16
   fast_tile_product<NB>(fp_smem, acc, k_len, w, rows,
       [&](int r) -> const __nv_bfloat16* {
         if (r >= rows) return nullptr;
-        return GLU ? x + (size_t)(sorted_pair[first + r] / top) * K : x + (size_t)(first + r) * K + k_first;
+        return GATHER ? x + (size_t)(sorted_pair[first + r] / top) * K : x + (size_t)(first + r) * K + k_first;
       },
       [&](int m, int n) -> const __nv_bfloat16* { return n0 + n < N ? we + ((size_t)m * N + n0 + n) * K : nullptr; });
   fast_tile_for_each<NB>(acc, [&](int r, int n, float v0, float v1) {
@@ -288,6 +316,9 @@ moe_product_fast_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16
     if constexpr (GLU) {
       const float pw = pair_w ? pair_w[sorted_pair[first + r]] : 1.f;
       ((__nv_bfloat16*)out_)[at] = __float2bfloat16_rn(moe_glu<__nv_bfloat16>(v0 * pw, v1 * pw, act));
+    } else if constexpr (MODE == MOE_ACT) {
+      const float pw = pair_w ? pair_w[sorted_pair[first + r]] : 1.f;
+      ((__nv_bfloat16*)out_)[at] = __float2bfloat16_rn(act_exact(v0 * pw, act));
     }
     else ((float*)out_)[(size_t)blockIdx.z * share_stride + at] = v0;
   });
@@ -295,19 +326,19 @@ moe_product_fast_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16
 
 static int moe_tiles(int P, int E, int BM = TP_BM) { return (P + BM - 1) / BM + (E < P ? E : P); }
 
-template <bool GLU>
+template <int MODE>
 static int moe_fast_launch(const void* x, const void* w, const int* offsets, const int* sorted_pair, void* out, int P, int E, int N,
                            int K, int top, int act, int shares, cudaStream_t stream, const float* pair_w = nullptr) {
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(moe_product_fast_kernel<GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, FP_SMEM_BYTES);
+    cudaError_t e = cudaFuncSetAttribute(moe_product_fast_kernel<MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, FP_SMEM_BYTES);
     if (e != cudaSuccess) QE_REFUSE("moe: shared memory: %s", cudaGetErrorString(e));
     configured = true;
   }
-  constexpr int BN = FpShape<GLU ? 2 : 1>::BN;
+  constexpr int BN = FpShape<MODE == MOE_GLU ? 2 : 1>::BN;
   dim3 grid(moe_tiles(P, E, FP_BM), (N + BN - 1) / BN, shares);
   const int k_share = shares > 1 ? ((K + shares - 1) / shares + FP_BK - 1) / FP_BK * FP_BK : K;
-  qe_launch(moe_product_fast_kernel<GLU>, grid, dim3(FP_THREADS), FP_SMEM_BYTES, stream, (const __nv_bfloat16*)x,
+  qe_launch(moe_product_fast_kernel<MODE>, grid, dim3(FP_THREADS), FP_SMEM_BYTES, stream, (const __nv_bfloat16*)x,
             (const __nv_bfloat16*)w, offsets, sorted_pair, out, E, N, K, top, act, k_share, (long)P * N, pair_w);
   return 0;
 }
@@ -319,18 +350,39 @@ extern "C" int qe_moe_gate_up(const void* x, const void* w, const int* offsets, 
                               int P, int E, int I, int K, int top, int act, int dtype, const float* pair_w, cudaStream_t stream) {
   if (P <= 0) return 0;
   if (moe_fast_applies(x, w, K, dtype)) {
-    if (int rc = moe_fast_launch<true>(x, w, offsets, sorted_pair, act_out, P, E, I, K, top, act, 1, stream, pair_w)) return rc;
+    if (int rc = moe_fast_launch<MOE_GLU>(x, w, offsets, sorted_pair, act_out, P, E, I, K, top, act, 1, stream, pair_w)) return rc;
     QE_CHECK_LAUNCH("moe_gate_up");
     return 0;
   }
   dim3 grid(moe_tiles(P, E), (I + TP_BN - 1) / TP_BN);
-#define MP(TT) qe_launch(moe_product_kernel<TT, true>, grid, dim3(TP_THREADS), 0, stream, (const TT*)x, (const TT*)w, offsets, \
+#define MP(TT) qe_launch(moe_product_kernel<TT, MOE_GLU>, grid, dim3(TP_THREADS), 0, stream, (const TT*)x, (const TT*)w, offsets, \
                          sorted_pair, act_out, E, I, K, top, act, pair_w)
   if (dtype == QE_DTYPE_F32) MP(float);
   else if (dtype == QE_DTYPE_BF16) MP(__nv_bfloat16);
   else QE_REFUSE("moe_gate_up: unknown dtype %d", dtype);
 #undef MP
   QE_CHECK_LAUNCH("moe_gate_up");
+  return 0;
+}
+
+// w [E, I, K]; act: the activation's code (common.cuh: act_for)
+extern "C" int qe_moe_up(const void* x, const void* w, const int* offsets, const int* sorted_pair, void* act_out, int P, int E,
+                         int I, int K, int top, int act, int dtype, const float* pair_w, cudaStream_t stream) {
+  if (P <= 0) return 0;
+  if (act < 0 || act > QE_ACT_MAX) QE_REFUSE("moe_up: unknown activation %d", act);
+  if (moe_fast_applies(x, w, K, dtype)) {
+    if (int rc = moe_fast_launch<MOE_ACT>(x, w, offsets, sorted_pair, act_out, P, E, I, K, top, act, 1, stream, pair_w)) return rc;
+    QE_CHECK_LAUNCH("moe_up");
+    return 0;
+  }
+  dim3 grid(moe_tiles(P, E), (I + TP_BN - 1) / TP_BN);
+#define MP(TT) qe_launch(moe_product_kernel<TT, MOE_ACT>, grid, dim3(TP_THREADS), 0, stream, (const TT*)x, (const TT*)w, offsets, \
+                         sorted_pair, act_out, E, I, K, top, act, pair_w)
+  if (dtype == QE_DTYPE_F32) MP(float);
+  else if (dtype == QE_DTYPE_BF16) MP(__nv_bfloat16);
+  else QE_REFUSE("moe_up: unknown dtype %d", dtype);
+#undef MP
+  QE_CHECK_LAUNCH("moe_up");
   return 0;
 }
 
@@ -348,14 +400,14 @@ extern "C" int qe_moe_down(const void* act_in, const void* w, const int* offsets
   if (P <= 0) return 0;
   if (shares < 1 || shares > 8) QE_REFUSE("moe_down: %d shares of K", shares);
   if (moe_fast_applies(act_in, w, K, dtype)) {
-    if (int rc = moe_fast_launch<false>(act_in, w, offsets, nullptr, (void*)y, P, E, N, K, 1, 0, shares, stream)) return rc;
+    if (int rc = moe_fast_launch<MOE_DOWN>(act_in, w, offsets, nullptr, (void*)y, P, E, N, K, 1, 0, shares, stream)) return rc;
     QE_CHECK_LAUNCH("moe_down");
     return 0;
   }
   // (the plain kernel adds up all of K: the other shares are zeros)
   if (shares > 1) cudaMemsetAsync(y + (size_t)P * N, 0, (size_t)(shares - 1) * P * N * sizeof(float), stream);
   dim3 grid(moe_tiles(P, E), (N + TP_BN - 1) / TP_BN);
-#define MP(TT) qe_launch(moe_product_kernel<TT, false>, grid, dim3(TP_THREADS), 0, stream, (const TT*)act_in, (const TT*)w, offsets, \
+#define MP(TT) qe_launch(moe_product_kernel<TT, MOE_DOWN>, grid, dim3(TP_THREADS), 0, stream, (const TT*)act_in, (const TT*)w, offsets, \
                          (const int*)nullptr, (void*)y, E, N, K, 1, 0, (const float*)nullptr)
   if (dtype == QE_DTYPE_F32) MP(float);
   else if (dtype == QE_DTYPE_BF16) MP(__nv_bfloat16);

@@ -118,6 +118,7 @@ class DecoderModel:
                 if geo not in geos:
                     geos.append(geo)
         self.attention_geometries = tuple(geos)
+        self.keeps_copy = any(b.keeps_copy for b in self.blocks)      # some layers read the stream rounded to the compute type
         self.capturable = all(getattr(b, "capturable", True) and getattr(b.mixer, "capturable", True) for b in self.blocks)
 
     # ---- what the cache manager and the loader ask --------------------------------------
@@ -191,7 +192,7 @@ class DecoderModel:
         [num_logit_rows, vocab] (None when no logits are wanted)."""
         lo = self.layout
         T, H = ctx.num_tokens, lo.hidden_size
-        stream = ops.ResidualStream.for_step(ctx.arena.alloc, T, H, ctx.dtype)
+        stream = ops.ResidualStream.for_step(ctx.arena.alloc, T, H, ctx.dtype, with_copy=self.keeps_copy)
         history = None
         if lo.layer_history:
             # the stream starts as entry 0 of the runs' results; a block that mixes them hands on ``mixed``
@@ -232,6 +233,8 @@ class DecoderModel:
             if history is not None:
                 history.run = i
             self.blocks[entry.layer].forward(ctx, stream, view, group, entry.write_cache)
+            if not self.blocks[entry.layer].keeps_copy:
+                stream.copy_current = False
         ctx.extras["next_cache"] = ctx.extras["weights_after_ffn"] = ctx.extras["norm_after_block"] = None
         if ctx.num_logit_rows == 0:
             return None

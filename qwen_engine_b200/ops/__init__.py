@@ -68,6 +68,16 @@ GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}     # the functions a gated feed-
 LIMITED_GLU = "swish_limit"    # ("swish_limit", L): g' = min(g, L), u' = clamp(u, -L, L), g' sigmoid(1.702 g') (u' + 1)
 
 
+ACTIVATIONS = {None: 0, "gelu_tanh": 1, "relu_squared": 2, "silu": 3}    # what a product may apply to its sums (feed-forwards without a gate)
+
+
+def activation_code(activation) -> int:
+    """The number the products take for the activation of their sums (0: none)."""
+    if activation not in ACTIVATIONS:
+        raise KernelRefused(f"unknown activation {activation!r}; known: {sorted(a for a in ACTIVATIONS if a)}")
+    return ACTIVATIONS[activation]
+
+
 def gate_activation_known(activation) -> bool:
     if isinstance(activation, (tuple, list)):
         return len(activation) == 2 and activation[0] == LIMITED_GLU and float(activation[1]) > 0.0
@@ -175,20 +185,22 @@ def prepare_matrix(w: torch.Tensor) -> torch.Tensor:
 
 
 def embedding(token_ids: torch.Tensor, table: torch.Tensor, out,
-              ssq: Optional[torch.Tensor] = None, scale: float = 1.0, accumulate: bool = False) -> None:
+              ssq: Optional[torch.Tensor] = None, scale: float = 1.0, accumulate: bool = False,
+              copy: Optional[torch.Tensor] = None) -> None:
     """out[t] = float32(table[token_ids[t]]) * scale; out is the float32 residual stream [T, H].  With ``ssq``
     [T, P] float32, ssq[t, 0] gets the row's sum of squares (one partial sum per row).  ``out`` may be a
     ``ResidualStream``: its rows are written and, if it keeps sums of squares, those too.
     ``accumulate``: the scaled rows are added to what the stream holds (its pending branch output stays
-    pending; sums of squares are no longer known)."""
+    pending; sums of squares are no longer known).  ``copy`` [T, H] in the table's dtype: the rows once more, rounded."""
     if isinstance(out, ResidualStream):
         stream = out
         if accumulate:
             embedding(token_ids, table, stream.resid, None, scale, True)
-            stream.n_ssq = 0
+            stream.n_ssq, stream.copy_current = 0, False
             return
-        embedding(token_ids, table, stream.resid, stream.ssq, scale)
+        embedding(token_ids, table, stream.resid, stream.ssq, scale, copy=stream.copy)
         stream.has_delta, stream.n_ssq = False, (1 if stream.ssq is not None else 0)
+        stream.copy_current = stream.copy is not None
         return
     _i32(token_ids, "token_ids")
     T, (V, H) = token_ids.numel(), table.shape
@@ -197,9 +209,12 @@ def embedding(token_ids: torch.Tensor, table: torch.Tensor, out,
     if ssq is not None:
         _need(ssq.dtype == torch.float32 and ssq.dim() == 2 and ssq.shape[0] == T and ssq.is_contiguous(),
               "embedding: ssq must be float32 [T, P]")
+    if copy is not None:
+        _need(copy.dtype == table.dtype and copy.shape == (T, H) and copy.is_contiguous() and not accumulate,
+              "embedding: the copy must be [T, H] in the table's dtype")
     _check(lib().qe_embedding(_ptr(token_ids), _ptr(table), _ptr(out), T, H, V, _dt(table), _ptr(ssq),
                               int(ssq.shape[1]) if ssq is not None else 0, ctypes.c_float(scale), int(bool(accumulate)),
-                              _stream()), "embedding")
+                              _ptr(copy), _stream()), "embedding")
 
 
 def add_rmsnorm(resid: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
@@ -240,23 +255,39 @@ class ResidualStream:
     into it at once (``ResidualSink``), or leaves it in ``delta`` [T, H] (compute dtype) with
     ``has_delta`` set, to be added by the next norm.  ``ssq`` [T, P] float32 holds ``n_ssq`` partial
     sums of squares of every row of ``resid`` when the kernel that last wrote the stream left them
-    (``n_ssq`` = 0: unknown); a norm fused into the next product starts from them."""
+    (``n_ssq`` = 0: unknown); a norm fused into the next product starts from them.
+    ``copy`` [T, H]: for arrangements whose sublayers read the stream itself, its rows rounded to the compute type
+    (None in float32, where the stream serves as it is), up to date while ``copy_current``: the kernels that write the
+    stream for such an arrangement leave it behind."""
 
-    def __init__(self, resid: torch.Tensor, delta: torch.Tensor, ssq: Optional[torch.Tensor] = None):
-        self.resid, self.delta, self.ssq = resid, delta, ssq
+    def __init__(self, resid: torch.Tensor, delta: torch.Tensor, ssq: Optional[torch.Tensor] = None,
+                 copy: Optional[torch.Tensor] = None):
+        self.resid, self.delta, self.ssq, self.copy = resid, delta, ssq, copy
         self.has_delta = False
         self.n_ssq = 0
+        self.copy_current = False
+
+    def rounded(self) -> torch.Tensor:
+        """The stream's rows in the compute type (the stream itself in float32)."""
+        if self.copy is None:
+            return self.resid
+        if not self.copy_current:
+            scaled_add(self.copy, self.resid, 1.0, first=True)
+            self.copy_current = True
+        return self.copy
 
     @classmethod
-    def for_step(cls, alloc, num_tokens: int, width: int, dtype: torch.dtype) -> "ResidualStream":
+    def for_step(cls, alloc, num_tokens: int, width: int, dtype: torch.dtype, with_copy: bool = False) -> "ResidualStream":
         """The stream of a step of ``num_tokens`` rows of ``width``, from ``alloc(shape, dtype)``.  For a few rows
         in bfloat16 it also gets room for the partial sums of squares that the products which add into the
         stream leave behind (one per 16 or per 8 columns, padded to whole float4s): their layout is the kernels'
-        business, so it is settled here, beside their fronts, and not by the model."""
+        business, so it is settled here, beside their fronts, and not by the model.  ``with_copy``: the stream keeps
+        its rows rounded to the compute type beside it (see ``copy``)."""
         ssq = None
         if dtype == torch.bfloat16 and num_tokens <= SMALL_M_MAX:
             ssq = alloc((num_tokens, -(-(-(-width // 8)) // 4) * 4), torch.float32)
-        return cls(alloc((num_tokens, width), torch.float32), alloc((num_tokens, width), dtype), ssq)
+        copy = alloc((num_tokens, width), dtype) if with_copy and dtype != torch.float32 else None
+        return cls(alloc((num_tokens, width), torch.float32), alloc((num_tokens, width), dtype), ssq, copy)
 
 
 class ResidualSink:
@@ -355,16 +386,18 @@ def splitk_splits(M: int, N: int, K: int, dtype: torch.dtype) -> int:
     return 0
 
 
-def linear_splitk(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: int, add: bool = False) -> None:
+def linear_splitk(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, splits: int, add: bool = False,
+                  activation: Optional[str] = None) -> None:
     """``linear`` in bfloat16 for up to 64 rows by clusters of ``splits`` CTAs that share 128 weight rows
     and meet through distributed shared memory; ``add``: out (float32) += the product."""
+    _need(not (add and activation), "linear_splitk: a product that is added to the stream has no activation")
     M, K = x.shape
     N = w.shape[0]
     _need(x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and w.shape == (N, K), "linear_splitk: bfloat16 operands, w [N, K]")
     _need(out.shape == (M, N) and out.dtype in (torch.bfloat16, torch.float32) and (not add or out.dtype == torch.float32),
           "linear_splitk: out must be [M, N], float32 to be added to")
     _need(x.is_contiguous() and w.is_contiguous() and out.is_contiguous(), "linear_splitk: operands must be contiguous")
-    mode = 2 if add else int(out.dtype == torch.float32)
+    mode = (2 if add else int(out.dtype == torch.float32)) | activation_code(activation) << 2
     _check(lib().qe_linear_tcgen05_splitk(_ptr(x), _ptr(w), _ptr(out), M, N, K, int(splits), mode, _stream()), "linear_splitk")
 
 
@@ -422,13 +455,16 @@ def _hand_over_next_weights() -> None:
         lib().qe_small_m_prefetch_next(_ptr(w), ctypes.c_ulonglong(w.numel() * w.element_size()))
 
 
-def linear(x, w: torch.Tensor, out: torch.Tensor) -> None:
+def linear(x, w: torch.Tensor, out: torch.Tensor, activation: Optional[str] = None) -> None:
     """out[M, N] = x[M, K] · w[N, K]^T, float32 accumulation; out in x's dtype or float32.
-    ``x`` may be a NormedInput (see there)."""
+    ``x`` may be a NormedInput (see there).  ``activation`` (``ACTIVATIONS``) is applied to the float32 sums in the
+    product's epilogue, whichever kernel serves it (not where ``out`` is a ResidualSink)."""
+    act = activation_code(activation)
     if isinstance(x, NormedInput):
-        if _linear_normed(x, w, out):
+        if not act and _linear_normed(x, w, out):
             return
         x = x.materialize()
+    _need(not (act and isinstance(out, ResidualSink)), "linear: a product that is added to the stream has no activation")
     if isinstance(out, ResidualSink):
         if _linear_into_stream(x, w, out, silu=False):
             return
@@ -438,21 +474,21 @@ def linear(x, w: torch.Tensor, out: torch.Tensor) -> None:
     _need(w.shape == (N, K) and w.dtype == x.dtype, f"linear: w {tuple(w.shape)} {w.dtype} does not fit x {tuple(x.shape)} {x.dtype}")
     _need(out.shape == (M, N) and out.dtype in (x.dtype, torch.float32), "linear: out must be [M, N] in x's dtype or float32")
     _need(x.is_contiguous() and w.is_contiguous() and out.is_contiguous(), "linear: operands must be contiguous")
-    out_f32 = int(out.dtype == torch.float32)
+    out_mode = int(out.dtype == torch.float32) | act << 1
     splits = splitk_splits(M, N, K, x.dtype)
     if splits:
-        linear_splitk(x, w, out, splits)
+        linear_splitk(x, w, out, splits, activation=activation)
         return
     if (x.dtype == torch.bfloat16 and SWAP_MIN_M <= M <= SMALL_M_MAX and N >= SWAP_MIN_N and K % 8 == 0
             and TCGEN05_ENABLED):
         # some tens of rows and many weight rows: the weights on the 128-row side of tcgen05.mma
-        _check(lib().qe_linear_tcgen05_swap(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_f32, _stream()), "linear")
+        _check(lib().qe_linear_tcgen05_swap(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_mode, _stream()), "linear")
         return
     if x.dtype == torch.bfloat16 and M <= SMALL_M_MAX and K % 8 == 0:
         # a few rows: stream every weight once through the tensor cores
         _hand_over_next_weights()
         lib().qe_small_m_rows8(int(SMALL_M_ROWS8))
-        _check(lib().qe_linear_small_m(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_f32, _stream()), "linear")
+        _check(lib().qe_linear_small_m(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_mode, _stream()), "linear")
         return
     if (x.dtype == torch.bfloat16 and TCGEN05_PAIRS and TCGEN05_ENABLED and K % 8 == 0
             and (-(-M // 256) * -(-N // 256) >= PAIR_MIN_TILES
@@ -460,13 +496,13 @@ def linear(x, w: torch.Tensor, out: torch.Tensor) -> None:
         # pairs of CTAs share a 256-row tile (tcgen05 cta_group::2): enough 256 x 256 tiles for every pair of SMs,
         # or the library's model of the kernels' times says so (fewer tiles: wide tiles all the same, or 2 or 4 pairs
         # per tile with a share of a long K each, meeting on chip)
-        linear_pairs(x, w, out)
+        linear_pairs(x, w, out, activation)
         return
     if x.dtype == torch.bfloat16 and M > SMALL_M_MAX and K % 8 == 0 and TCGEN05_ENABLED:
         # many rows: TMA-fed tcgen05 tensor cores with the accumulator in tensor memory
-        _check(lib().qe_linear_tcgen05(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_f32, _stream()), "linear")
+        _check(lib().qe_linear_tcgen05(_ptr(x), _ptr(w), _ptr(out), M, N, K, out_mode, _stream()), "linear")
         return
-    _check(lib().qe_linear_generic(_ptr(x), _ptr(w), _ptr(out), M, N, K, _dt(x), out_f32, _stream()), "linear")
+    _check(lib().qe_linear_generic(_ptr(x), _ptr(w), _ptr(out), M, N, K, _dt(x), out_mode, _stream()), "linear")
 
 
 PAIR_PLAN = True        # products of many rows with fewer than PAIR_MIN_TILES tiles go where the library's model of the kernels' times sends them
@@ -483,7 +519,7 @@ def pair_k_splits(M: int, N: int, K: int) -> int:
     return int(lib().qe_pair_k_splits(int(M), int(N), int(K), 0))
 
 
-def linear_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
+def linear_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, activation: Optional[str] = None) -> None:
     """``linear`` in bfloat16 by the kernel in which two CTAs share a 256-row tile; any number of rows
     (few tiles: 256 x 128 tiles; ``linear`` itself comes here only for large products)."""
     M, K = x.shape
@@ -492,8 +528,8 @@ def linear_pairs(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
           "linear_pairs: bfloat16 operands with K a multiple of 8")
     _need(out.shape == (M, N) and out.dtype in (torch.bfloat16, torch.float32), "linear_pairs: out must be [M, N]")
     _need(x.is_contiguous() and w.is_contiguous() and out.is_contiguous(), "linear_pairs: operands must be contiguous")
-    _check(lib().qe_linear_tcgen05_pair(_ptr(x), _ptr(w), _ptr(out), M, N, K, int(out.dtype == torch.float32), _stream()),
-           "linear_pairs")
+    _check(lib().qe_linear_tcgen05_pair(_ptr(x), _ptr(w), _ptr(out), M, N, K,
+                                        int(out.dtype == torch.float32) | activation_code(activation) << 1, _stream()), "linear_pairs")
 
 
 def swiglu_fused_applies(M: int, I: int, K: int, dtype: torch.dtype) -> bool:
@@ -1095,7 +1131,8 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
     ``softcap`` > 0: the scaled score s becomes softcap tanh(s / softcap).  ``sinks`` (float32 [Hq]): exp(sinks[h])
     joins the softmax's denominator of head h; it has no key and no value.  ``value_shift`` s: the weights of a head
     whose kv head is c meet the values of kv head (c + s) mod Hkv (a mixer that mixes the heads' weights sums such
-    outputs).  Every kernel takes the three (not together with a distance bias or a cache of one plane).
+    outputs).  Every kernel takes the three (not together with a distance bias; over a cache of
+    one plane bent scores and sinks only).
     ``value_shifts`` S > 1: out is [S, T, Hq D] and entry s is the output for shift s; where the whole step is served by
     the kernels for few rows, the shifts are one launch (a grid dimension), else one launch each.
 
@@ -1130,8 +1167,8 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
     if sinks is not None:
         _need(sinks.dtype == torch.float32 and sinks.numel() == Hq and sinks.is_contiguous(), "paged_attention: sinks must be float32 [Hq]")
     if plain:
-        _need(planes == 2 and slopes is None and 0 <= value_shift < Hkv,
-              "paged_attention: bent scores, sinks and shifted values go with a cache of two planes and no distance bias")
+        _need(slopes is None and 0 <= value_shift < Hkv, "paged_attention: bent scores, sinks and shifted values go without a distance bias")
+        _need(planes == 2 or (value_shift == 0 and S == 1), "paged_attention: shifted values go with a cache of two planes")
     if planes == 1:
         _need(slopes is None, "paged_attention: no distance bias over a cache of one plane")
         key = index.get((Hq, Hkv, D, window, False, 1))
@@ -1344,7 +1381,7 @@ def head_norm_gate(x: torch.Tensor, gate: Optional[torch.Tensor], weight: Option
         _stream()), "head_norm_gate")
 
 
-def latent_prepare(down: torch.Tensor, q: torch.Tensor, norm_w: torch.Tensor, eps: float, positions: torch.Tensor,
+def latent_prepare(down: Optional[torch.Tensor], q: torch.Tensor, norm_w: Optional[torch.Tensor], eps: float, positions: torch.Tensor,
                    inv_freq: torch.Tensor, rot_dims: int, cache: torch.Tensor, slot_mapping: torch.Tensor,
                    qlat: torch.Tensor, num_heads: int, plain_dim: int, latent_dim: int, rot_dim: int,
                    write_kv: bool = True) -> None:
@@ -1352,29 +1389,37 @@ def latent_prepare(down: torch.Tensor, q: torch.Tensor, norm_w: torch.Tensor, ep
     first R channels are RMS-normed (weight ``norm_w``) into the token's cache row, the last Dr are the key part all
     heads share, whose first ``rot_dims`` channels turn (pairs (i, i + rot_dims / 2), angle position x inv_freq[i]) on
     their way into the cache row's tail.  ``q`` [T, H (dn + Dr)]: every head's last Dr channels turn likewise into
-    ``qlat`` [T, H, R + Dr] behind the room for the head's folded plain part.  cache [pages, 1, 1, page, R + Dr]."""
-    _rows(down, "latent_prepare: down")
+    ``qlat`` [T, H, R + Dr] behind the room for the head's folded plain part.  cache [pages, 1, 1, page, R + Dr].
+    Without ``write_kv`` (a layer that reads another layer's cache) only the queries' parts turn; ``down`` and ``norm_w``
+    may then be None."""
     _rows(q, "latent_prepare: q")
     T = q.shape[0]
     H, dn, R, Dr = num_heads, plain_dim, latent_dim, rot_dim
-    _need(down.shape == (T, R + Dr) and q.shape == (T, H * (dn + Dr)) and down.dtype == q.dtype == qlat.dtype == cache.dtype,
-          "latent_prepare: down [T, R + Dr], q [T, H (dn + Dr)] in the cache's dtype")
+    _need(q.shape == (T, H * (dn + Dr)) and q.dtype == qlat.dtype == cache.dtype, "latent_prepare: q [T, H (dn + Dr)] in the cache's dtype")
+    if write_kv:
+        _need(down is not None and norm_w is not None, "latent_prepare: a cache write needs the latent and its norm's weight")
+        _rows(down, "latent_prepare: down")
+        _need(down.shape == (T, R + Dr) and down.dtype == q.dtype, "latent_prepare: down must be [T, R + Dr] in the cache's dtype")
+        _need(norm_w.dtype == torch.float32 and norm_w.shape == (R,), "latent_prepare: the norm weight must be float32 [R]")
+    else:
+        down = norm_w = None
     _need(qlat.shape == (T, H * (R + Dr)) and qlat.is_contiguous(), "latent_prepare: qlat must be [T, H (R + Dr)]")
     _need(cache.dim() == 5 and cache.shape[1] == 1 and cache.shape[2] == 1 and cache.shape[4] == R + Dr and cache.is_contiguous(),
           "latent_prepare: cache must be [pages, 1, 1, page, R + Dr]")
-    _need(norm_w.dtype == torch.float32 and norm_w.shape == (R,) and inv_freq.dtype == torch.float32
-          and inv_freq.numel() >= rot_dims // 2, "latent_prepare: float32 norm weight [R] and inv_freq [rot_dims / 2]")
+    _need(inv_freq.dtype == torch.float32 and inv_freq.numel() >= rot_dims // 2, "latent_prepare: inv_freq must be float32 [rot_dims / 2]")
     _i32(positions, "positions")
     _i32(slot_mapping, "slot_mapping")
-    _check(lib().qe_latent_prepare(_ptr(down), ctypes.c_long(down.stride(0)), _ptr(q), ctypes.c_long(q.stride(0)), _ptr(norm_w),
+    _check(lib().qe_latent_prepare(_ptr(down), ctypes.c_long(down.stride(0) if down is not None else 0), _ptr(q), ctypes.c_long(q.stride(0)), _ptr(norm_w),
                                    ctypes.c_float(eps), _ptr(positions), _ptr(inv_freq), int(rot_dims), _ptr(cache),
                                    _ptr(slot_mapping), _ptr(qlat), T, H, dn, R, Dr, int(bool(write_kv)), _dt(q), _stream()),
            "latent_prepare")
 
 
-def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stride: int, out_head_stride: int) -> None:
+def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stride: int, out_head_stride: int,
+                gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h * out_head_stride + n] = sum_k w[h, n, k] x[t, h * x_head_stride + k]: one matrix per head, w [H, N, K];
-    x and out are rows (unit stride along columns) in w's dtype, float32 accumulation."""
+    x and out are rows (unit stride along columns) in w's dtype, float32 accumulation.  ``gate`` [T, H] in w's dtype (rows
+    may be strided): the sums of head h are multiplied by sigmoid(gate[t, h]) before they are rounded."""
     _rows(x, "head_linear: x")
     _rows(out, "head_linear: out")
     H, N, K = w.shape
@@ -1382,9 +1427,12 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stri
     _need(w.is_contiguous() and x.dtype == w.dtype == out.dtype and out.shape[0] == M, "head_linear: operands of one dtype, w contiguous")
     _need((H - 1) * x_head_stride + K <= x.shape[1] and (H - 1) * out_head_stride + N <= out.shape[1],
           "head_linear: the heads do not fit the rows")
+    if gate is not None:
+        _rows(gate, "head_linear: gate")
+        _need(gate.shape == (M, H) and gate.dtype == w.dtype, "head_linear: gate must be [T, H] in w's dtype")
     _check(lib().qe_head_linear(_ptr(x), ctypes.c_long(x.stride(0)), ctypes.c_long(x_head_stride), _ptr(w), _ptr(out),
-                                ctypes.c_long(out.stride(0)), ctypes.c_long(out_head_stride), M, H, N, K, _dt(x), _stream()),
-           "head_linear")
+                                ctypes.c_long(out.stride(0)), ctypes.c_long(out_head_stride), M, H, N, K, _dt(x), _ptr(gate),
+                                ctypes.c_long(gate.stride(0) if gate is not None else 0), _stream()), "head_linear")
 
 
 def short_conv(x: torch.Tensor, w: torch.Tensor, state: torch.Tensor, ctx, out: torch.Tensor, write_state: bool = True,
@@ -1452,33 +1500,40 @@ def delta_rule_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: Option
            "delta_rule_scan")
 
 
-ROUTER_SCORINGS = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2}
+ROUTER_SCORINGS = {"softmax_chosen": 0, "softmax_all": 1, "sigmoid": 2, "sigmoid_sum": 3}
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], top_idx: torch.Tensor, top_w: torch.Tensor,
-              scoring: str = "softmax_chosen", correction: Optional[torch.Tensor] = None) -> None:
+              scoring: str = "softmax_chosen", correction: Optional[torch.Tensor] = None, weight_scale: float = 1.0,
+              n_always: int = 0) -> None:
     """Router of routed experts: z = w x[t] + bias in float32 (x in the compute type, w float32 [E, W]).
     ``softmax_chosen``: the ``top`` largest logits' experts into top_idx int32 [T, top] (the lower index wins a tie)
     and the softmax over those logits alone into top_w float32 [T, top].
     ``softmax_all``: s = softmax(z) over all E outputs; the ``top`` largest of s + correction (float32 [E], optional)
     are chosen, and their weights are their s as it is (not made to sum to one).
-    ``sigmoid``: every output is scored alone, s = sigmoid(z); the ``top`` largest are chosen and their weights are their s."""
+    ``sigmoid``: every output is scored alone, s = sigmoid(z); the ``top`` largest are chosen and their weights are their s.
+    ``sigmoid_sum``: as before, the chosen s divided by their sum (+ 1e-20) and multiplied by ``weight_scale``.
+    ``n_always`` S > 0: w has a last row more and the outputs S columns more: behind its chosen experts every token names
+    E .. E + S - 1 (the pieces of an expert that every token uses), each with the weight sigmoid(w[E] x[t])."""
     T, W = x.shape
-    E = w.shape[0]
-    top = top_idx.shape[1]
+    S = int(n_always)
+    E = w.shape[0] - int(S > 0)
+    top = top_idx.shape[1] - S
+    _need(weight_scale == 1.0 or scoring == "sigmoid_sum", "moe_route: a scale of the weights goes with sigmoid_sum")
+    _need(S == 0 or bias is None, "moe_route: no bias beside experts that every token uses")
     _need(scoring in ROUTER_SCORINGS, f"moe_route: unknown scoring {scoring!r}; known: {sorted(ROUTER_SCORINGS)}")
-    _need(x.is_contiguous() and w.dtype == torch.float32 and w.shape == (E, W) and w.is_contiguous(), "moe_route: w must be float32 [E, W]")
+    _need(x.is_contiguous() and w.dtype == torch.float32 and w.dim() == 2 and w.shape[1] == W and w.is_contiguous(), "moe_route: w must be float32 [E, W]")
     _need(bias is None or (bias.dtype == torch.float32 and bias.shape == (E,)), "moe_route: bias must be float32 [E]")
     _need(correction is None or (correction.dtype == torch.float32 and correction.shape == (E,) and correction.is_contiguous()
                                  and scoring == "softmax_all"), "moe_route: correction must be float32 [E], with softmax_all")
-    _need(top_idx.shape == (T, top) and top_idx.dtype == torch.int32 and top_idx.is_contiguous()
-          and top_w.shape == (T, top) and top_w.dtype == torch.float32 and top_w.is_contiguous(), "moe_route: outputs [T, top]")
+    _need(top >= 1 and top_idx.shape[0] == T and top_idx.dtype == torch.int32 and top_idx.is_contiguous()
+          and top_w.shape == top_idx.shape and top_w.dtype == torch.float32 and top_w.is_contiguous(), "moe_route: outputs [T, top]")
     _check(lib().qe_moe_route(_ptr(x), _ptr(w), _ptr(bias), _ptr(top_idx), _ptr(top_w), T, W, E, top, _dt(x),
-                              ROUTER_SCORINGS[scoring], _ptr(correction), _stream()), "moe_route")
+                              ROUTER_SCORINGS[scoring], _ptr(correction), ctypes.c_float(weight_scale), S, _stream()), "moe_route")
 
 
 def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                out: torch.Tensor, activation, alloc, num_identity: int = 0, weight_inputs: bool = False) -> None:
+                out: torch.Tensor, activation, alloc, num_identity: int = 0, weight_inputs: bool = False, gated: bool = True) -> None:
     """out[t] = sum_j top_w[t, j] * W_down[e] glu(W_gate[e] x[t], W_up[e] x[t]) with e = top_idx[t, j]: the pairs are
     ordered by expert on the device, each expert's rows run as tiles of two grouped products, and the token's choices
     are summed in their order.  w_gate_up [E, 2 I, K] (gate rows, then up rows), w_down [E, N, I]; ``alloc(shape,
@@ -1486,12 +1541,14 @@ def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_g
     ``num_identity``: top_idx may also name E .. E + num_identity - 1, experts without weights whose output is
     x[t] itself (N = K then); their pairs are ordered behind the others and only the weighted sum looks at them.
     ``weight_inputs``: the weight multiplies what the expert reads, not what it returns: out[t] = sum_j expert_e(top_w[t, j]
-    x[t]).  The first products are linear, so the weight meets their float32 sums ahead of the activation."""
+    x[t]).  The first products are linear, so the weight meets their float32 sums ahead of the activation.
+    ``gated`` False: experts without a gate, W_down[e] f(W_up[e] x[t]) with w_gate_up [E, I, K] their up matrices and
+    ``activation`` one of ``ACTIVATIONS``."""
     T, K = x.shape
     E, I2, _ = w_gate_up.shape
-    I, N, top = I2 // 2, w_down.shape[1], top_idx.shape[1]
+    I, N, top = (I2 // 2 if gated else I2), w_down.shape[1], top_idx.shape[1]
     P = T * top
-    _need(x.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_gate_up.shape == (E, 2 * I, K)
+    _need(x.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_gate_up.shape == (E, (2 if gated else 1) * I, K)
           and w_down.shape == (E, N, I) and x.dtype == w_gate_up.dtype == w_down.dtype, "moe_experts: w_gate_up [E, 2 I, K], w_down [E, N, I] in x's dtype")
     _need(out.shape == (T, N) and out.is_contiguous(), "moe_experts: out must be [T, N]")
     _need(num_identity >= 0 and (num_identity == 0 or N == K), "moe_experts: identity experts need outputs of the input's width")
@@ -1501,8 +1558,10 @@ def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_g
     place = alloc((P,), torch.int32)
     _check(lib().qe_moe_sort(_ptr(top_idx), _ptr(offsets), _ptr(sorted_pair), _ptr(place), P, E + num_identity, _stream()), "moe_sort")
     act = alloc((P, I), x.dtype)
-    _check(lib().qe_moe_gate_up(_ptr(x), _ptr(w_gate_up), _ptr(offsets), _ptr(sorted_pair), _ptr(act), P, E, I, K, top,
-                                gate_code(activation), _dt(x), _ptr(top_w if weight_inputs else None), _stream()), "moe_gate_up")
+    first = lib().qe_moe_gate_up if gated else lib().qe_moe_up
+    _check(first(_ptr(x), _ptr(w_gate_up), _ptr(offsets), _ptr(sorted_pair), _ptr(act), P, E, I, K, top,
+                 gate_code(activation) if gated else activation_code(activation), _dt(x), _ptr(top_w if weight_inputs else None),
+                 _stream()), "moe_gate_up")
     # a few rows (decoded tokens): the down product cuts K into shares so that enough CTAs pull the weights; the shares' sums
     # are added, in their order, where the token's choices are
     shares = int(lib().qe_moe_down_shares(P, I, _dt(x)))

@@ -9,12 +9,13 @@ from .latent_attention import LatentAttention
 from .delta_rule import GatedDeltaRule
 from .moe import RoutedExperts
 from .parallel import ParallelMixers
-from .mlp import SwiGLU
+from .mlp import MLP, SwiGLU
 from .block import PreNormBlock
 from .gated_post_norm import GatedPostNormBlock
 from .sandwich_norm import SandwichNormBlock
+from .post_norm import PostNormBlock
 
 __all__ = ["Arena", "Block", "FeedForward", "GroupStepView", "Mixer", "Norm", "Part", "PartSpec",
            "PositionEncoding", "StepContext", "register", "NORMS", "POSITION_ENCODINGS", "MIXERS",
-           "FEED_FORWARDS", "BLOCKS", "RMSNorm", "GroupRMSNorm", "NeoxRope", "ScaledRope", "GQAAttention", "GatedLinearAttention", "DecayedLinearAttention", "LatentAttention", "GatedDeltaRule", "RoutedExperts", "ParallelMixers", "SwiGLU",
-           "PreNormBlock", "GatedPostNormBlock", "SandwichNormBlock"]
+           "FEED_FORWARDS", "BLOCKS", "RMSNorm", "GroupRMSNorm", "NeoxRope", "ScaledRope", "GQAAttention", "GatedLinearAttention", "DecayedLinearAttention", "LatentAttention", "GatedDeltaRule", "RoutedExperts", "ParallelMixers", "SwiGLU", "MLP",
+           "PreNormBlock", "GatedPostNormBlock", "SandwichNormBlock", "PostNormBlock"]

@@ -316,6 +316,7 @@ class FeedForward(Part):
 class Block(Part):
     mixer: Mixer
     capturable = True             # False if any of its parts says so: steps of the model are then never graph-captured
+    keeps_copy = False            # True if the block reads the stream's rounded copy and leaves it up to date (ops.ResidualStream.copy)
 
     def cache_specs(self) -> list:
         """Every cache a run of the layer keeps: its mixer's, and behind them whatever the arrangement itself keeps

@@ -79,3 +79,40 @@ class SwiGLU(FeedForward):
             ops.act_mul(gate_up, act, self.activation)
             ops.linear(act, self.w_down, out)
         ops.prefetch_next(None)
+
+
+@register("feed_forward", "mlp")
+class MLP(FeedForward):
+    """A feed-forward without a gate: down(f(up(x))), no biases; ``activation`` is one of ``ops.ACTIVATIONS`` and is applied
+    to the up product's float32 sums in its epilogue, whichever kernel serves it."""
+
+    writes_through_linear = True  # out is the out of the last product
+    takes_lazy_input = True       # x goes to one product only
+
+    def __init__(self, hidden_size: int, intermediate_size: int, activation: str = "gelu_tanh", names: tuple = ("up", "down")):
+        if activation not in ops.ACTIVATIONS or not activation:
+            raise ValueError(f"unknown activation {activation!r}; known: {sorted(a for a in ops.ACTIVATIONS if a)}")
+        self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
+        self.activation, self.names = activation, tuple(names)
+        self.w_up = self.w_down = None
+
+    def weight_specs(self, prefix: str) -> list[WeightSpec]:
+        up, down = self.names
+        return [WeightSpec(prefix + up, (self.intermediate_size, self.hidden_size), MATRIX),
+                WeightSpec(prefix + down, (self.hidden_size, self.intermediate_size), MATRIX)]
+
+    def load(self, prefix, source, dtype, device) -> None:
+        up, down = self.names
+        self.w_up = ops.prepare_matrix(source.get(prefix + up).to(dtype).to(device))
+        self.w_down = ops.prepare_matrix(source.get(prefix + down).to(dtype).to(device))
+
+    def first_weights(self):
+        return self.w_up
+
+    def forward(self, ctx: StepContext, x, out) -> None:
+        act = ctx.arena.alloc((ctx.num_tokens, self.intermediate_size), ctx.dtype)
+        ops.prefetch_next(self.w_down)
+        ops.linear(x, self.w_up, act, activation=self.activation)
+        ops.prefetch_next(step_hint(ctx, "weights_after_ffn"))
+        ops.linear(act, self.w_down, out)
+        ops.prefetch_next(None)

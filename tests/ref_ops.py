@@ -21,18 +21,21 @@ def prepare_matrix(w):
     return w.contiguous()
 
 
-def embedding(token_ids, table, out, ssq=None, scale=1.0, accumulate=False):
+def embedding(token_ids, table, out, ssq=None, scale=1.0, accumulate=False, copy=None):
     from qwen_engine_b200.ops import ResidualStream
     if isinstance(out, ResidualStream):
         if not accumulate:
             out.has_delta = False
         out.n_ssq = 0
+        copy, out.copy_current = (None, False) if accumulate else (out.copy, out.copy is not None)
         out = out.resid
     rows = table[token_ids.long()].to(torch.float32) * scale
     if accumulate:
         out.add_(rows)
     else:
         out.copy_(rows)
+        if copy is not None:
+            copy.copy_(rows.to(copy.dtype))
 
 
 def _rms(x, weight, eps):
@@ -55,13 +58,27 @@ def add_rmsnorm_rows(resid, delta, rows, weight, eps, out):
     out.copy_(_rms(x, weight, eps).to(out.dtype))
 
 
-def linear(x, w, out):
+def activation_of(z, activation):
+    """z float32 -> f(z) for the activations a product may apply to its sums."""
+    import math
+    if activation is None:
+        return z
+    if activation == "relu_squared":
+        return torch.clamp(z, min=0.0) ** 2
+    if activation == "gelu_tanh":
+        return 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
+    if activation == "silu":
+        return z * torch.sigmoid(z)
+    raise ValueError(activation)
+
+
+def linear(x, w, out, activation=None):
     from qwen_engine_b200.ops import NormedInput, ResidualSink
     if isinstance(x, NormedInput):
         x = x.materialize()
     if isinstance(out, ResidualSink):
         out = out.as_delta()
-    out.copy_((x.to(torch.float32) @ w.to(torch.float32).t()).to(out.dtype))
+    out.copy_(activation_of(x.to(torch.float32) @ w.to(torch.float32).t(), activation).to(out.dtype))
 
 
 def _rotate(x, positions, inv_freq, rotary_dim, magnitude=1.0):
@@ -282,11 +299,14 @@ def latent_prepare(down, q, norm_w, eps, positions, inv_freq, rot_dims, cache, s
     out[:, :, R:] = turn(q.reshape(T, H, dn + Dr)[:, :, dn:]).to(qlat.dtype)
 
 
-def head_linear(x, w, out, x_head_stride, out_head_stride):
+def head_linear(x, w, out, x_head_stride, out_head_stride, gate=None):
     H, N, K = w.shape
     for h in range(H):
         xs = x[:, h * x_head_stride:h * x_head_stride + K].to(torch.float32)
-        out[:, h * out_head_stride:h * out_head_stride + N] = (xs @ w[h].to(torch.float32).t()).to(out.dtype)
+        y = xs @ w[h].to(torch.float32).t()
+        if gate is not None:
+            y = y * torch.sigmoid(gate[:, h:h + 1].to(torch.float32))
+        out[:, h * out_head_stride:h * out_head_stride + N] = y.to(out.dtype)
 
 
 def short_conv(x, w, state, ctx, out, write_state=True, silu=True):
@@ -344,8 +364,14 @@ def delta_rule_scan(q, k, v, g, beta, state, ctx, out, num_heads, num_key_heads,
             state[slots[r]] = S
 
 
-def moe_route(x, w, bias, top_idx, top_w, scoring="softmax_chosen", correction=None):
+def moe_route(x, w, bias, top_idx, top_w, scoring="softmax_chosen", correction=None, weight_scale=1.0, n_always=0):
     z = x.to(torch.float32) @ w.t()
+    if n_always:                        # the router's last row weighs the experts that every token uses
+        E = w.shape[0] - 1
+        k = top_idx.shape[1] - n_always
+        top_idx[:, k:] = torch.arange(E, E + n_always, dtype=torch.int32)
+        top_w[:, k:] = torch.sigmoid(z[:, E:])
+        z, top_idx, top_w = z[:, :E], top_idx[:, :k], top_w[:, :k]
     if bias is not None:
         z = z + bias
     if scoring == "softmax_all":
@@ -356,13 +382,18 @@ def moe_route(x, w, bias, top_idx, top_w, scoring="softmax_chosen", correction=N
         return
     val, idx = torch.topk(z, top_idx.shape[1], dim=-1)
     top_idx.copy_(idx.to(torch.int32))
+    if scoring == "sigmoid_sum":
+        s = torch.sigmoid(val)
+        top_w.copy_(s / (s.sum(dim=-1, keepdim=True) + 1e-20) * weight_scale)
+        return
     top_w.copy_(torch.sigmoid(val) if scoring == "sigmoid" else torch.softmax(val, dim=-1))
 
 
-def moe_experts(x, top_idx, top_w, w_gate_up, w_down, out, activation, alloc, num_identity=0, weight_inputs=False):
+def moe_experts(x, top_idx, top_w, w_gate_up, w_down, out, activation, alloc, num_identity=0, weight_inputs=False,
+                gated=True):
     T = x.shape[0]
     E = w_gate_up.shape[0]
-    I = w_gate_up.shape[1] // 2
+    I = w_gate_up.shape[1] // 2 if gated else w_gate_up.shape[1]
     acc = torch.zeros(T, w_down.shape[1], dtype=torch.float32)
     for t in range(T):
         for j in range(top_idx.shape[1]):
@@ -374,9 +405,11 @@ def moe_experts(x, top_idx, top_w, w_gate_up, w_down, out, activation, alloc, nu
             gu = x[t:t + 1].to(torch.float32) @ w_gate_up[e].to(torch.float32).t()
             if weight_inputs:                # the weight meets the first products' sums ahead of the activation
                 gu = gu * float(top_w[t, j])
-            gu = gu.to(x.dtype)
-            act = torch.empty(1, I, dtype=x.dtype)
-            act_mul(gu, act, activation)
+            if gated:
+                act = torch.empty(1, I, dtype=x.dtype)
+                act_mul(gu.to(x.dtype), act, activation)
+            else:
+                act = activation_of(gu, activation).to(x.dtype)
             acc[t] += (1.0 if weight_inputs else float(top_w[t, j])) * (act.to(torch.float32) @ w_down[e].to(torch.float32).t())[0]
     out.copy_(acc.to(out.dtype))
 
