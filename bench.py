@@ -527,6 +527,21 @@ def pufivik_config_of(sz: dict) -> dict:
                 embedding=dict(scale=1.0), residual_mult=0.5, layers=four * (sz["layers"] // 4))
 
 
+def zugunex_config_of(sz: dict) -> dict:
+    """A Zugunex model at the sizes of ``sz``: latent attention in every layer (the latent and head sizes of the Besavik
+    model's), every second layer reading the latent of the one before it; windows of ``window`` tokens; a dense
+    feed-forward in the first layer and eight experts of half its width, two per token, beside a shared expert of that
+    same width, in the others."""
+    D = sz["head_dim"]
+    own = dict(heads=sz["heads"], dim=D, rot_dim=D // 2, vdim=D, kv_rank=D + D // 2, scale=(D + D // 2) ** -0.5,
+               mask=dict(size=sz["window"]), rot=dict(base=1000000.0, dims=D // 2))
+    dense = dict(kind="dense", ff=sz["ff"])
+    moe = dict(kind="moe", expert=dict(ff=sz["ff"] // 2), router=dict(experts=8, top=2, scale=1.0), shared=dict(ff=sz["ff"] // 2))
+    layers = [dict(type="latent_attention", mixer=own if i % 2 == 0 else dict(own, kv_from=i - 1), mlp=dense if i == 0 else moe)
+              for i in range(sz["layers"])]
+    return dict(architecture="Zugunex", vocab=sz["vocab"], width=sz["width"], norm=dict(eps=1e-6), layers=layers)
+
+
 def pufivik_kernels_alone(torch, ops, peaks) -> dict:
     """The kernels and kernel options that Pufivik adds, each alone on rows that do not fit in L2 (16 384 tokens of width
     2 048: a float32 stream of 134 MB), beside the like kernel of the other models on the same rows: device time (CUDA
@@ -729,7 +744,7 @@ def compare_designs(args) -> int:
     bfloat16), and the device time of every class of operation in one eager step of each (CUDA events around every
     call, the calls of a class added up).  ``--compare besavik``: a Besavik model beside both.  ``--compare merudra``: a
     Merudra model beside a Besavik and a Qwen3 model.  ``--compare pufivik``: a Pufivik model beside a Merudra and a Qwen3
-    model.  Prints one JSON line."""
+    model.  ``--compare zugunex``: a Zugunex model beside a Besavik and a Qwen3 model.  Prints one JSON line."""
     import torch
     from qwen_engine_b200 import ops
     from qwen_engine_b200.config import preset_config_dict
@@ -841,12 +856,14 @@ def compare_designs(args) -> int:
             out[name]["pufivik"] = measure(config_from_dict(pufivik_config_of(sz)), "pufivik")
         if args.compare in ("merudra", "pufivik"):
             out[name]["merudra"] = measure(config_from_dict(merudra_config_of(sz)), "merudra")
-        if args.compare in ("besavik", "merudra"):
+        if args.compare == "zugunex":
+            out[name]["zugunex"] = measure(config_from_dict(zugunex_config_of(sz)), "zugunex")
+        if args.compare in ("besavik", "merudra", "zugunex"):
             out[name]["besavik"] = measure(config_from_dict(besavik_config_of(sz)), "besavik")
-        if args.compare not in ("merudra", "pufivik"):
+        if args.compare not in ("merudra", "pufivik", "zugunex"):
             out[name]["ganidra"] = measure(config_from_dict(ganidra_config_of(sz)), "ganidra")
         out[name]["qwen3"] = measure(config_from_dict(qraw), "qwen3")
-        designs = [d for d in ("pufivik", "merudra", "besavik", "ganidra", "qwen3") if d in out[name]]
+        designs = [d for d in ("zugunex", "pufivik", "merudra", "besavik", "ganidra", "qwen3") if d in out[name]]
         for other in designs[1:]:
             g, q = out[name][designs[0]], out[name][other]
             out[name][f"{designs[0]}_over_{other}"] = {"prefill": round(g["prefill"]["tokens_per_s"] / q["prefill"]["tokens_per_s"], 3),
@@ -856,7 +873,7 @@ def compare_designs(args) -> int:
         alone = (merudra_kernels_alone if args.compare == "merudra" else pufivik_kernels_alone)(torch, ops, peaks)
     clocks.stop()
     title = {"besavik": "Besavik beside Ganidra and Qwen3", "merudra": "Merudra beside Besavik and Qwen3",
-             "pufivik": "Pufivik beside Merudra and Qwen3"}.get(args.compare, "Ganidra beside Qwen3")
+             "pufivik": "Pufivik beside Merudra and Qwen3", "zugunex": "Zugunex beside Besavik and Qwen3"}.get(args.compare, "Ganidra beside Qwen3")
     print(json.dumps({"metric": f"prefill and decode tok/s, {title} at equal sizes", "impl": "ours", "n_gpus": 1,
                       "dtype": "bf16", "data": "synthetic: uniform random token ids, random weights N(0, 0.02) seed 2",
                       "steps": args.steps, "warmup": args.warmup, "peaks": peaks_src, "sizes": out,
@@ -885,9 +902,9 @@ def main() -> int:
     ap.add_argument("--no-kernels", action="store_true", help="skip the per-kernel-class timings")
     ap.add_argument("--profile", choices=["decode", "prefill"], default=None,
                     help="bracket that timed region with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--compare", choices=["ganidra", "besavik", "merudra", "pufivik"], default=None,
+    ap.add_argument("--compare", choices=["ganidra", "besavik", "merudra", "pufivik", "zugunex"], default=None,
                     help="instead of the default workload: prefill and decode of a Ganidra model beside a Qwen3 model of equal "
-                         "sizes (besavik: a Besavik model beside both; merudra: a Merudra model beside a Besavik and a Qwen3 model; pufivik: a Pufivik model beside a Merudra and a Qwen3 model), with the device time of every class of operation "
+                         "sizes (besavik: a Besavik model beside both; merudra: a Merudra model beside a Besavik and a Qwen3 model; pufivik: a Pufivik model beside a Merudra and a Qwen3 model; zugunex: a Zugunex model beside a Besavik and a Qwen3 model), with the device time of every class of operation "
                          "(one JSON line)")
     ap.add_argument("--compare-size", choices=sorted(COMPARE_SIZES), default=None, help="with --compare: one size only")
     args = ap.parse_args()
