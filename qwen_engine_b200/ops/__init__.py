@@ -51,6 +51,8 @@ DECODE_ATTENTION_MMA_EARLY = True   # that kernel requests earlier steps' keys b
 DECODE_ATTENTION_MMA_BESIDE_TC = True   # also for the decoded tokens of a step whose prompt portions go to the tcgen05 kernel
 SHIFTS_IN_ONE_LAUNCH = True          # a mixer that mixes its heads' weights: the shifts of the values' kv head as one launch where the step has no long portion
 DECODE_ATTENTION_MMA_WIDE = True    # steps with at most as many attention CTAs as SMs: CTAs of 8 warps, one per SM (and contexts split for 148 CTAs, not 296)
+LATENT_DECODE = True                 # decoded tokens over a latent cache (one plane, one kv head): the kernel whose warps stream key groups of their own
+LATENT_DECODE_MIN_PART = 128         # keys of a part at least where a step's contexts are cut for that kernel
 DECODE_PREFETCH_KV_MB = 12          # that kernel asks L2 for the next layer's keys and values when a layer's are at most this many MB (0: never).  Measured (0.6B, context 1 024, asked for before the kernel's dependency wait): 4.4 MB (one request) 0.698 -> 0.690 ms a step, 8.8 MB 0.777 -> 0.765, 17.6 MB equal, 35 MB (eight) 0.915 -> 0.957
 TC_ROWS = 256           # rows per work item of the tcgen05 attention kernel (two halves of 128)
 TC_BN = 128             # keys per step of the tcgen05 attention kernel
@@ -769,7 +771,7 @@ class DeviceWaitTimeout(RuntimeError):
 
 
 _STATUS_WORDS = ("qe_gemm_tc", "qe_gemm_tc_swap", "qe_gemm_tc_pair", "qe_gemm_tc_splitk", "qe_flash_attention_tc",
-                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m")
+                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode")
 
 
 def device_status() -> dict[str, int]:
@@ -1065,6 +1067,16 @@ def decode_splits(num_reqs: int, max_tokens: int, geometries, dtype: torch.dtype
         Hq, Hkv, D, window, _ = split_geometry(geo)
         span = min(max_tokens, window) if window else max_tokens
         target = FLASH_TARGET_CTAS
+        if latent_decode_supported(geo, dtype):
+            # one CTA per SM; the parts of a request form a cluster (as many of 8, 4, 2 as fit on chip, keep every CTA on the
+            # GPU at once and leave each part enough keys)
+            most, tiles = int(lib().qe_latent_decode_max_parts(D)), -(-Hq // 16)
+            parts = 1
+            while (parts * 2 <= most and num_reqs * tiles * parts * 2 <= TC_TARGET_CTAS and span >= parts * 2 * LATENT_DECODE_MIN_PART
+                   and (parts * 2 < 8 or num_reqs * tiles * 8 <= 64)):
+                parts *= 2
+            out[geo] = parts
+            continue
         if (DECODE_ATTENTION_MMA and DECODE_ATTENTION_MMA_WIDE and dtype == torch.bfloat16 and D == 128
                 and Hq // Hkv <= 16 and num_reqs * Hkv <= TC_TARGET_CTAS):
             target = TC_TARGET_CTAS                                       # one CTA of 8 warps per SM
@@ -1104,6 +1116,14 @@ def _merge_counters(device, kernel: str = "fa") -> torch.Tensor:
     return t
 
 
+def latent_decode_supported(geo, dtype: torch.dtype) -> bool:
+    """Whether ``qe_latent_decode`` takes this geometry's decoded tokens: bfloat16, one plane and one kv head of up to 256
+    channels, at most as many heads as the flash kernel's items hold rows."""
+    Hq, Hkv, D, _, biased = split_geometry(geo)
+    return (LATENT_DECODE and dtype == torch.bfloat16 and geometry_planes(geo) == 1 and Hkv == 1 and D % 16 == 0 and D <= 256
+            and Hq <= FLASH_ROWS and not biased)
+
+
 def _decode_mma_serves(plan, key, qkv: torch.Tensor, Hq: int, Hkv: int, D: int) -> bool:
     """Whether the step's requests that are not on the tcgen05 kernel (geometry index ``key`` of the plan) go to
     the tensor-core kernel for decoded tokens: items of at most 16 rows, head size 128."""
@@ -1121,7 +1141,7 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
                     out: torch.Tensor, scale: float, window: int, num_heads: int, num_kv_heads: int,
                     head_dim: int, next_pages: Optional[torch.Tensor] = None,
                     slopes: Optional[torch.Tensor] = None, softcap: float = 0.0, sinks: Optional[torch.Tensor] = None,
-                    value_shift: int = 0, value_shifts: int = 1) -> None:
+                    value_shift: int = 0, value_shifts: int = 1, value_dim: Optional[int] = None) -> None:
     """Attention of the step's queries (the q part of qkv [T, (Hq+2Hkv) D]) over the keys and values
     of their requests in ``kv_pages``; out [T, Hq D].  ``ctx`` is the StepContext (cu_q, ctx_lens,
     the plan that ``plan_attention`` made, and the arena for the parts of split contexts).
@@ -1135,6 +1155,8 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
     one plane bent scores and sinks only).
     ``value_shifts`` S > 1: out is [S, T, Hq D] and entry s is the output for shift s; where the whole step is served by
     the kernels for few rows, the shifts are one launch (a grid dimension), else one launch each.
+    ``value_dim`` (a cache of one plane): only so many of a key's first channels are its value; what the output holds
+    behind them is not defined.
 
     ``next_pages``: the cache of the layer that runs after this one, if it has the same shape (the same
     pages at the same places): a decode step's kernel may ask L2 for that layer's keys and values."""
@@ -1202,6 +1224,20 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
             part_acc = ctx.arena.alloc((S * n_parts * Hkv * part_rows, D), torch.float32)
             part_ml = ctx.arena.alloc((S * n_parts * Hkv * part_rows, 2), torch.float32)
         counters = _merge_counters(qkv.device) if 0 < S * n_parts * Hkv <= _MERGE_COUNTERS else None
+        _need(value_dim is None or (planes == 1 and 1 <= value_dim <= D), "paged_attention: a value size of its own goes with a cache of one plane")
+        if (planes == 1 and softcap <= 0.0 and latent_decode_supported((Hq, Hkv, D, window, False, 1), qkv.dtype)
+                and (max_rows <= 16 or ctx.max_q_len == 1) and qkv.stride(0) % 8 == 0
+                and n_parts * -(-max_rows // 16) <= _MERGE_COUNTERS):
+            # decoded tokens over a latent cache: every warp streams key groups of its own, values out of the same rows
+            last_attention_kernel = "latent_decode"
+            cluster = int(same_parts) if n_items == n_parts else 0
+            if cluster > int(lib().qe_latent_decode_max_parts(D)):
+                cluster = 0
+            _check(lib().qe_latent_decode(
+                _ptr(qkv), ctypes.c_long(qkv.stride(0)), _ptr(kv_pages), _ptr(block_tables), int(block_tables.shape[1]), _ptr(items), n_items,
+                _ptr(out), _ptr(part_acc), _ptr(part_ml), int(part_rows), _ptr(_merge_counters(qkv.device)), int(max_rows), cluster,
+                ctypes.c_float(scale), int(window), Hq, D, int(value_dim or D), int(kv_pages.shape[3]), _ptr(sinks), _stream()), "latent_decode")
+            return
         # every request in the same few parts: the parts of a request form a cluster and meet on chip
         cluster = int(same_parts) if DECODE_ATTENTION_CLUSTERS and n_items == n_parts else 0
         if _decode_mma_serves(plan, key, qkv, Hq, Hkv, D):

@@ -182,7 +182,8 @@ class LatentAttention(Mixer):
                            view.slot_mapping, qlat, H, dn, R, dr, write_kv=writes)
         ops.head_linear(q, self.w_uk_t, qlat, dn + dr, D)
         olat = ctx.arena.alloc((T, H * D), ctx.dtype)
-        ops.paged_attention(qlat, cache, view.block_tables, ctx, olat, self.scale, self.window or 0, H, 1, D, sinks=self.sinks)
+        ops.paged_attention(qlat, cache, view.block_tables, ctx, olat, self.scale, self.window or 0, H, 1, D, sinks=self.sinks,
+                            value_dim=R)
         gate = proj[:, self.gate_at:self.gate_at + (H if self.output_gate == "sigmoid_head" else self.gate_width)] if self.output_gate else None
         per_head = self.output_gate == "sigmoid_head"
         elementwise = self.output_gate == "sigmoid" or scale != 1.0

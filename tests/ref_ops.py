@@ -152,7 +152,7 @@ def plan_attention(q_lens, ctx_lens, page_size, geometries=(), dtype=None, unifo
 
 
 def paged_attention(qkv, kv_pages, block_tables, ctx, out, scale, window, num_heads, num_kv_heads, head_dim, next_pages=None,
-                    slopes=None, softcap=0.0, sinks=None, value_shift=0, value_shifts=1):
+                    slopes=None, softcap=0.0, sinks=None, value_shift=0, value_shifts=1, value_dim=None):
     """For each request: gather its keys and values from the pages by its block table, then
     softmax(scale q k^T + mask) v with key j allowed for the query at position i iff
     j <= i and (window == 0 or j > i - window)."""
