@@ -1568,6 +1568,14 @@ def moe_route(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], to
                               ROUTER_SCORINGS[scoring], _ptr(correction), ctypes.c_float(weight_scale), S, _stream()), "moe_route")
 
 
+MOE_SMALL_MAX_T = 64     # tokens up to which experts without a gate go through the weight-streaming products
+
+
+def moe_small_applies(T: int, I: int, K: int, dtype: torch.dtype) -> bool:
+    """Whether the products of experts without a gate are served by the kernels that stream every used weight once."""
+    return dtype == torch.bfloat16 and 1 <= T <= MOE_SMALL_MAX_T and K % 8 == 0 and I % 8 == 0
+
+
 def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                 out: torch.Tensor, activation, alloc, num_identity: int = 0, weight_inputs: bool = False, gated: bool = True) -> None:
     """out[t] = sum_j top_w[t, j] * W_down[e] glu(W_gate[e] x[t], W_up[e] x[t]) with e = top_idx[t, j]: the pairs are
@@ -1594,6 +1602,15 @@ def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_g
     place = alloc((P,), torch.int32)
     _check(lib().qe_moe_sort(_ptr(top_idx), _ptr(offsets), _ptr(sorted_pair), _ptr(place), P, E + num_identity, _stream()), "moe_sort")
     act = alloc((P, I), x.dtype)
+    if not gated and moe_small_applies(T, I, K, x.dtype):
+        _check(lib().qe_moe_small_up(_ptr(x), _ptr(w_gate_up), _ptr(offsets), _ptr(sorted_pair), _ptr(act), T, P, E, I, K, top,
+                                     activation_code(activation), _ptr(top_w if weight_inputs else None), _stream()), "moe_small_up")
+        y = alloc((1, P, N), torch.float32)
+        _check(lib().qe_moe_small_down(_ptr(act), _ptr(w_down), _ptr(offsets), _ptr(y), T, P, E, N, I, _stream()), "moe_small_down")
+        _check(lib().qe_moe_combine(_ptr(y), _ptr(place), _ptr(None if weight_inputs else top_w), _ptr(out), T, N, top, 1, _dt(out),
+                                    _ptr(top_idx if num_identity else None), E, _ptr(x if num_identity else None), _dt(x), _stream()),
+               "moe_combine")
+        return
     first = lib().qe_moe_gate_up if gated else lib().qe_moe_up
     _check(first(_ptr(x), _ptr(w_gate_up), _ptr(offsets), _ptr(sorted_pair), _ptr(act), P, E, I, K, top,
                  gate_code(activation) if gated else activation_code(activation), _dt(x), _ptr(top_w if weight_inputs else None),
