@@ -771,7 +771,7 @@ class DeviceWaitTimeout(RuntimeError):
 
 
 _STATUS_WORDS = ("qe_gemm_tc", "qe_gemm_tc_swap", "qe_gemm_tc_pair", "qe_gemm_tc_splitk", "qe_flash_attention_tc",
-                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode")
+                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode", "qe_moe_tc")
 
 
 def device_status() -> dict[str, int]:
@@ -1576,6 +1576,14 @@ def moe_small_applies(T: int, I: int, K: int, dtype: torch.dtype) -> bool:
     return dtype == torch.bfloat16 and 1 <= T <= MOE_SMALL_MAX_T and K % 8 == 0 and I % 8 == 0
 
 
+MOE_TC_MIN_PAIRS = 513   # (token, choice) pairs from which they go through the grouped tcgen05 products
+
+
+def moe_tc_applies(P: int, I: int, K: int, N: int, dtype: torch.dtype) -> bool:
+    """Whether the products of experts without a gate are served by the grouped tcgen05 kernel: bfloat16, many pairs."""
+    return TCGEN05_ENABLED and dtype == torch.bfloat16 and P >= MOE_TC_MIN_PAIRS and K % 8 == 0 and I % 8 == 0
+
+
 def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
                 out: torch.Tensor, activation, alloc, num_identity: int = 0, weight_inputs: bool = False, gated: bool = True) -> None:
     """out[t] = sum_j top_w[t, j] * W_down[e] glu(W_gate[e] x[t], W_up[e] x[t]) with e = top_idx[t, j]: the pairs are
@@ -1608,6 +1616,18 @@ def moe_experts(x: torch.Tensor, top_idx: torch.Tensor, top_w: torch.Tensor, w_g
         y = alloc((1, P, N), torch.float32)
         _check(lib().qe_moe_small_down(_ptr(act), _ptr(w_down), _ptr(offsets), _ptr(y), T, P, E, N, I, _stream()), "moe_small_down")
         _check(lib().qe_moe_combine(_ptr(y), _ptr(place), _ptr(None if weight_inputs else top_w), _ptr(out), T, N, top, 1, _dt(out),
+                                    _ptr(top_idx if num_identity else None), E, _ptr(x if num_identity else None), _dt(x), _stream()),
+               "moe_combine")
+        return
+    if not gated and not weight_inputs and moe_tc_applies(P, I, K, N, x.dtype):
+        # many pairs: the rows in the experts' order, then both products on the tensor cores' tiles
+        xs = alloc((P, K), x.dtype)
+        _check(lib().qe_moe_gather(_ptr(x), _ptr(sorted_pair), _ptr(xs), P, K, top, _stream()), "moe_gather")
+        _check(lib().qe_moe_tc(_ptr(xs), _ptr(w_gate_up), _ptr(offsets), _ptr(act), P, E, I, K, activation_code(activation), 1, _stream()),
+               "moe_tc")
+        y = alloc((1, P, N), torch.float32)
+        _check(lib().qe_moe_tc(_ptr(act), _ptr(w_down), _ptr(offsets), _ptr(y), P, E, N, I, 0, 0, _stream()), "moe_tc")
+        _check(lib().qe_moe_combine(_ptr(y), _ptr(place), _ptr(top_w), _ptr(out), T, N, top, 1, _dt(out),
                                     _ptr(top_idx if num_identity else None), E, _ptr(x if num_identity else None), _dt(x), _stream()),
                "moe_combine")
         return

@@ -318,6 +318,38 @@ def test_experts_without_a_gate_beside_a_shared_one(ops, dtype, W, ff, E, top, s
     assert ops.device_status() == {}
 
 
+@pytest.mark.parametrize("W,ff,counts", [(64, 40, [0, 1, 127, 128, 129, 256, 0, 300]), (128, 264, [513]), (520, 72, [0, 0, 640, 3]),
+                                         (8, 8, [600, 1]), (256, 512, [130] * 40)])
+def test_grouped_products_of_many_rows_at_the_tiles_borders(ops, W, ff, counts):
+    """Experts whose rows fill tiles exactly, miss them by one, or are none; one choice a token, so a row is one expert's."""
+    from qwen_engine_b200.parts.base import Arena
+    g = torch.Generator().manual_seed(W + ff)
+    E, T = len(counts), sum(counts)
+    idx = torch.tensor([e for e, n in enumerate(counts) for _ in range(n)])[torch.randperm(T, generator=g)]
+    x = torch.randn(T, W, generator=g).to(BF16)
+    up = (torch.randn(E, ff, W, generator=g) / math.sqrt(W)).to(BF16)
+    down = (torch.randn(E, W, ff, generator=g) / math.sqrt(ff)).to(BF16)
+    wgt = torch.rand(T, 1, generator=g) + 0.5
+    assert ops.moe_tc_applies(T, ff, W, W, BF16)
+    outs = []
+    for tc in (True, False):
+        out = torch.full((T, W), float("nan"), dtype=BF16, device=DEV)
+        saved, ops.MOE_TC_MIN_PAIRS = ops.MOE_TC_MIN_PAIRS, (1 if tc else 1 << 30)
+        try:
+            ops.moe_experts(x.to(DEV), idx.to(torch.int32)[:, None].contiguous().to(DEV), wgt.to(DEV), up.to(DEV), down.to(DEV), out, "relu_squared",
+                            Arena(DEV, 1 << 24).alloc, gated=False)
+        finally:
+            ops.MOE_TC_MIN_PAIRS = saved
+        outs.append(out)
+    want = torch.empty(T, W, dtype=F64)
+    for e in range(E):
+        at = idx == e
+        want[at] = wgt.double()[at] * (plain.relu_squared(x[at].double() @ up[e].double().T) @ down[e].double().T)
+    for out in outs:
+        _close(out, want, BF16, "grouped", tol=2e-2)
+    assert ops.device_status() == {}
+
+
 # ---- the mixer through its cache ---------------------------------------------------------------------------------------------
 class _Dict:
     def __init__(self, d):
