@@ -54,6 +54,8 @@ DECODE_ATTENTION_MMA_WIDE = True    # steps with at most as many attention CTAs 
 LATENT_DECODE = True                 # decoded tokens over a latent cache (one plane, one kv head): the kernel whose warps stream key groups of their own
 LATENT_DECODE_MIN_PART = 128         # keys of a part at least where a step's contexts are cut for that kernel
 DECODE_PREFETCH_KV_MB = 12          # that kernel asks L2 for the next layer's keys and values when a layer's are at most this many MB (0: never).  Measured (0.6B, context 1 024, asked for before the kernel's dependency wait): 4.4 MB (one request) 0.698 -> 0.690 ms a step, 8.8 MB 0.777 -> 0.765, 17.6 MB equal, 35 MB (eight) 0.915 -> 0.957
+LATENT_TC = True        # prompt portions over a latent cache on tcgen05
+LATENT_TC_ROWS = 128    # rows (query token x head) per work item of that kernel
 TC_ROWS = 256           # rows per work item of the tcgen05 attention kernel (two halves of 128)
 TC_BN = 128             # keys per step of the tcgen05 attention kernel
 TC_MIN_ROWS = 65        # rows of a request's portion from which the tcgen05 kernel serves it
@@ -771,7 +773,7 @@ class DeviceWaitTimeout(RuntimeError):
 
 
 _STATUS_WORDS = ("qe_gemm_tc", "qe_gemm_tc_swap", "qe_gemm_tc_pair", "qe_gemm_tc_splitk", "qe_flash_attention_tc",
-                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode", "qe_moe_tc")
+                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode", "qe_moe_tc", "qe_latent_attention_tc")
 
 
 def device_status() -> dict[str, int]:
@@ -1004,7 +1006,8 @@ def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
             continue
         G = Hq // Hkv
         tpt = FLASH_ROWS // G
-        use_tc = uniform_splits is None and geometry_planes(geo) == 2 and tc_attention_supported(dtype, Hq, Hkv, D, page_size)
+        latent_tc = latent_tc_supported(geo, dtype, page_size)
+        use_tc = uniform_splits is None and (latent_tc or (geometry_planes(geo) == 2 and tc_attention_supported(dtype, Hq, Hkv, D, page_size)))
         on_tc = [use_tc and n * G >= TC_MIN_ROWS for n in q_lens]
         tc_tiles: list = []
         base = sum(-(-n // tpt) for n, tc in zip(q_lens, on_tc) if not tc) * Hkv
@@ -1015,7 +1018,7 @@ def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
         for r, (n, c) in enumerate(zip(q_lens, ctx_lens)):
             total = c + n
             if on_tc[r]:
-                tc_tpt = TC_ROWS // G
+                tc_tpt = (LATENT_TC_ROWS if latent_tc else TC_ROWS) // G
                 for q0 in range(0, n, tc_tpt):
                     lo = max(0, c + q0 - window + 1) if window else 0
                     hi = c + min(n, q0 + tc_tpt)
@@ -1048,7 +1051,12 @@ def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
         sizes = {m for m in merge[3::4]}
         same = sizes.pop() if len(sizes) == 1 and not whole else 0
         plan[f"fa{gi}_info"] = [n_parts, part_rows, int(max_rows <= 16), max_rows, same if same in (2, 4, 8) else 0]
-        if tc_tiles:
+        if tc_tiles and latent_tc:
+            # a tile's keys are not cut: the tiles alone, those with the most keys first
+            tc_tiles.sort(key=lambda t: -t[0])
+            plan[f"tc{gi}_items"] = [x for _, lo, hi, (r, q0, first, n, c) in tc_tiles for x in (r, q0, lo, hi, -1, 0, 0, first, n, c, 0, 0)]
+            plan[f"tc{gi}_info"] = [0, LATENT_TC_ROWS, len(tc_tiles)]
+        elif tc_tiles:
             tc_items, tc_parts, tc_sched, tc_ctas = _plan_tc_tiles(tc_tiles, Hkv)
             plan[f"tc{gi}_items"] = tc_items
             plan[f"tc{gi}_sched"] = tc_sched
@@ -1114,6 +1122,14 @@ def _merge_counters(device, kernel: str = "fa") -> torch.Tensor:
         t = torch.zeros(_MERGE_COUNTERS, dtype=torch.int32, device=device)
         _merge_counter_tensors[key] = t
     return t
+
+
+def latent_tc_supported(geo, dtype: torch.dtype, page_size: int) -> bool:
+    """Whether the tcgen05 kernel for latent caches takes this geometry's prompt portions: bfloat16, one plane and one kv
+    head of up to 256 channels, up to 128 heads, pages a power of two of at least 8 tokens."""
+    Hq, Hkv, D, _, biased = split_geometry(geo)
+    return (LATENT_TC and dtype == torch.bfloat16 and geometry_planes(geo) == 1 and Hkv == 1 and D % 16 == 0 and D <= 256
+            and Hq <= FLASH_ROWS and not biased and page_size >= 8 and page_size & (page_size - 1) == 0)
 
 
 def latent_decode_supported(geo, dtype: torch.dtype) -> bool:
@@ -1196,7 +1212,16 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
         key = index.get((Hq, Hkv, D, window, False, 1))
     else:
         key = index.get((Hq, Hkv, D, window, True)) if slopes is not None else index.get((Hq, Hkv, D, window), index.get((Hq, Hkv, D, window, False)))
-    if key is not None and f"tc{key}_items" in plan:
+    _need(value_dim is None or (planes == 1 and 1 <= value_dim <= D), "paged_attention: a value size of its own goes with a cache of one plane")
+    if key is not None and f"tc{key}_items" in plan and planes == 1:
+        _need(qkv.is_contiguous() and softcap <= 0.0, "paged_attention: over latents, contiguous queries and scores as they are")
+        last_attention_kernel = "latent_attention_tc"
+        tc_items = plan[f"tc{key}_items"]
+        _check(lib().qe_latent_attention_tc(
+            _ptr(qkv), T, _ptr(kv_pages), int(kv_pages.shape[0]), _ptr(block_tables), int(block_tables.shape[1]), _ptr(tc_items),
+            tc_items.numel() // FLASH_ITEM_INTS, _ptr(out), ctypes.c_float(scale), int(window), Hq, D, int(value_dim or D),
+            int(kv_pages.shape[3]), _ptr(sinks), _stream()), "latent_attention_tc")
+    elif key is not None and f"tc{key}_items" in plan:
         last_attention_kernel = "flash_attention_tc"
         tc_items = plan[f"tc{key}_items"]
         tc_parts, tc_rows, tc_ctas = plan[f"tc{key}_info_host"]
@@ -1224,7 +1249,6 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
             part_acc = ctx.arena.alloc((S * n_parts * Hkv * part_rows, D), torch.float32)
             part_ml = ctx.arena.alloc((S * n_parts * Hkv * part_rows, 2), torch.float32)
         counters = _merge_counters(qkv.device) if 0 < S * n_parts * Hkv <= _MERGE_COUNTERS else None
-        _need(value_dim is None or (planes == 1 and 1 <= value_dim <= D), "paged_attention: a value size of its own goes with a cache of one plane")
         if (planes == 1 and softcap <= 0.0 and latent_decode_supported((Hq, Hkv, D, window, False, 1), qkv.dtype)
                 and (max_rows <= 16 or ctx.max_q_len == 1) and qkv.stride(0) % 8 == 0
                 and n_parts * -(-max_rows // 16) <= _MERGE_COUNTERS):
