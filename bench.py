@@ -653,6 +653,133 @@ def pufivik_kernels_alone(torch, ops, peaks) -> dict:
     return {"rows": T, "width": W, "kernels": out}
 
 
+def zugunex_kernels_alone(torch, ops, peaks) -> dict:
+    """The kernels and kernel options that Zugunex adds, each alone beside its like among the other models' kernels on the same
+    rows: device time (CUDA events around three replays of a graph of ten launches); for passes over rows the bytes moved over the measured copy
+    rate, for products and attention the multiply-adds over the measured bfloat16 rate, for decoded tokens the bytes of
+    the weights or keys over the copy rate.  Inputs larger than L2 where the operation is a pass over rows."""
+    from types import SimpleNamespace
+    from qwen_engine_b200.engine.runner import ModelRunner
+    from qwen_engine_b200.parts.base import Arena
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    hbm, tflops = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"])
+    g = torch.Generator(device=dev).manual_seed(6)
+    rnd = lambda *shape, dtype=f32, std=1.0: (torch.randn(*shape, device=dev, dtype=f32, generator=g) * std).to(dtype)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    out: dict = {}
+
+    def timed(name, fn, nbytes=None, flops=None, like=None):
+        for _ in range(3):
+            fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()               # ten launches from a graph: the host's time for a call is not measured
+        with torch.cuda.graph(graph):
+            for _ in range(10):
+                fn()
+        graph.replay()
+        torch.cuda.synchronize()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        for _ in range(3):
+            graph.replay()
+        b.record()
+        torch.cuda.synchronize()
+        us = a.elapsed_time(b) * 1000.0 / 30.0
+        rec = {"us": round(us, 1)}
+        if nbytes:
+            rec.update(mb=round(nbytes / 1e6, 1), gbs=round(nbytes / us / 1e3, 1), frac_of_copy=round(nbytes / us / 1e3 / hbm, 3))
+        if flops:
+            rec.update(tflops=round(flops / us / 1e6, 1), frac_of_bf16=round(flops / us / 1e6 / tflops, 3))
+        if like:
+            rec["like"] = like
+        out[name] = rec
+
+    T, W = 16384, 2048
+    stream, branch, copy, wt = rnd(T, W), rnd(T, W, dtype=bf), torch.empty(T, W, device=dev, dtype=bf), rnd(W) + 1.0
+    timed("gated_norm_add without gate, with the rounded copy", lambda: ops.gated_norm_add(stream, branch, None, None, wt, 1e-6, stream, copy),
+          T * W * 12, like="add_rmsnorm")
+    timed("add_rmsnorm", lambda: ops.add_rmsnorm(stream, branch, wt, 1e-6, copy), T * W * 12)
+    E, top = 8, 2
+    ti, tw = torch.empty(T, top + 1, device=dev, dtype=torch.int32), torch.empty(T, top + 1, device=dev, dtype=f32)
+    ti2, tw2 = torch.empty(T, top, device=dev, dtype=torch.int32), torch.empty(T, top, device=dev, dtype=f32)
+    rw, rw2 = rnd(E + 1, W, std=0.05), rnd(E, W, std=0.05)
+    timed("moe_route, sigmoids that sum to one, shared expert's gate", lambda: ops.moe_route(branch, rw, None, ti, tw, "sigmoid_sum", n_always=1),
+          T * W * 2, like="moe_route over the chosen")
+    timed("moe_route over the chosen", lambda: ops.moe_route(branch, rw2, None, ti2, tw2, "softmax_chosen"), T * W * 2)
+    del stream, copy
+    H, dn, dr, dv, R, page = 16, 128, 64, 128, 192, 16
+    D = R + dr
+    n = 4096
+    olat, w_uv, gate = rnd(n, H * D, dtype=bf), rnd(H, dv, R, dtype=bf, std=0.05), rnd(n, H, dtype=bf)
+    inner = torch.empty(n, H * dv, device=dev, dtype=bf)
+    head_flops = 2 * n * H * R * dv
+    timed("head_linear with a gate per head", lambda: ops.head_linear(olat, w_uv, inner, D, dv, gate=gate), flops=head_flops, like="head_linear")
+    timed("head_linear", lambda: ops.head_linear(olat, w_uv, inner, D, dv), flops=head_flops)
+    xa, up, act = rnd(2048, W, dtype=bf), rnd(6144, W, dtype=bf, std=0.02), torch.empty(2048, 6144, device=dev, dtype=bf)
+    for label, a in (("linear with gelu", "gelu_tanh"), ("linear with the square of relu", "relu_squared"), ("linear", None)):
+        timed(label + ", 2 048 x 6 144 x 2 048", lambda: ops.linear(xa, up, act, activation=a), flops=2 * 2048 * 6144 * W, like="linear" if a else None)
+    xd, ad = xa[:8].contiguous(), torch.empty(8, 6144, device=dev, dtype=bf)
+    for label, a in (("linear with gelu", "gelu_tanh"), ("linear", None)):
+        timed(label + ", 8 rows", lambda: ops.linear(xd, up, ad, activation=a), nbytes=6144 * W * 2, like="linear" if a else None)
+    # experts: 2 048 tokens and 8, two of eight experts of 3 072 channels; beside the gated experts of the other models
+    I = 3072
+    w1, w1g, w2 = rnd(E, I, W, dtype=bf, std=0.02), rnd(E, 2 * I, W, dtype=bf, std=0.02), rnd(E, W, I, dtype=bf, std=0.02)
+    arena = Arena(dev, 1 << 29)
+    for t in (2048, 8):
+        x = xa[:t].contiguous()
+        idx = torch.stack([torch.randperm(E, device=dev, generator=g)[:top] for _ in range(t)]).to(torch.int32)
+        wgt, res = torch.full((t, top), 0.5, device=dev), torch.empty(t, W, device=dev, dtype=bf)
+
+        def run(w, gated, a):
+            m = arena.mark()
+            ops.moe_experts(x, idx, wgt, w, w2, res, a, arena.alloc, gated=gated)
+            arena.release(m)
+        many = t > 64
+        for label, w, gated, a, like in ((f"experts without a gate, {t} tokens", w1, False, "relu_squared", f"gated experts, {t} tokens"),
+                                         (f"gated experts, {t} tokens", w1g, True, "silu", None)):
+            mats = 3 if gated else 2
+            timed(label, lambda: run(w, gated, a), flops=2 * t * top * I * W * mats if many else None,
+                  nbytes=None if many else int(idx.unique().numel()) * I * W * 2 * mats, like=like)
+    del w1, w1g, w2, arena
+    # attention over latents, window 1 024: four prompts of 2 048 tokens; and 64 decoded tokens behind 1 024 keys each
+    window = 1024
+    sinks = rnd(H)
+    for kind, q_lens, ctx_lens in (("prompts", [2048] * 4, [0] * 4), ("decoded tokens", [1] * 8, [2047] * 8), ("decoded tokens, 64 requests", [1] * 64, [2047] * 64)):
+        reqs, t = len(q_lens), sum(q_lens)
+        blocks = 2048 // page
+        pages = rnd(reqs * blocks, 1, 1, page, D, dtype=bf)
+        tables = torch.arange(reqs * blocks, device=dev, dtype=torch.int32).view(reqs, blocks).contiguous()
+        qlat, res = rnd(t, H * D, dtype=bf), torch.empty(t, H * D, device=dev, dtype=bf)
+        cu = [0]
+        for m in q_lens:
+            cu.append(cu[-1] + m)
+        geo = (H, 1, D, window, False, 1)
+        pairs = sum(min(c + i + 1, window) for m, c in zip(q_lens, ctx_lens) for i in range(m))
+        prompts = kind == "prompts"
+        for label, own in (("the kernel for latents", True), ("the flash kernel", False)):
+            saved = ops.LATENT_TC, ops.LATENT_DECODE
+            ops.LATENT_TC = ops.LATENT_DECODE = own
+            try:
+                splits = None if prompts else ops.decode_splits(reqs, 2048, (geo,), bf)
+                plan = ops.plan_attention(q_lens, ctx_lens, page, (geo,), bf, uniform_splits=splits)
+                devplan = ModelRunner._device_plan(plan, {"plan_" + k: i32(v) for k, v in plan.items()}, (geo,))
+                actx = SimpleNamespace(cu_q=i32(cu), ctx_lens=i32(ctx_lens), q_lens_host=q_lens, ctx_lens_host=ctx_lens, attn_plan=devplan,
+                                       max_q_len=max(q_lens), arena=Arena(dev, 1 << 28))
+
+                def attend():
+                    m = actx.arena.mark()
+                    ops.paged_attention(qlat, pages, tables, actx, res, D ** -0.5, window, H, 1, D, sinks=sinks, value_dim=R)
+                    actx.arena.release(m)
+                name = f"attention over latents, {kind}, {label}"
+                timed(name, attend, flops=2 * pairs * H * (D + R) if prompts else None, nbytes=None if prompts else reqs * window * D * 2,
+                      like=f"attention over latents, {kind}, the flash kernel" if own else None)
+                out[name]["kernel"] = ops.last_attention_kernel
+            finally:
+                ops.LATENT_TC, ops.LATENT_DECODE = saved
+    ops.check_device_status()
+    return {"rows": T, "width": W, "kernels": out}
+
+
 def merudra_kernels_alone(torch, ops, peaks) -> dict:
     """The kernels that Merudra's arrangement adds, each alone on rows that do not fit in L2 (16 384 tokens of width
     2 048: a float32 stream of 134 MB), beside the like kernel of the other models on the same rows: device time (CUDA
@@ -869,8 +996,9 @@ def compare_designs(args) -> int:
             out[name][f"{designs[0]}_over_{other}"] = {"prefill": round(g["prefill"]["tokens_per_s"] / q["prefill"]["tokens_per_s"], 3),
                                                       "decode": round(g["decode"]["tokens_per_s"] / q["decode"]["tokens_per_s"], 3)}
     alone = None
-    if not args.compare_size and args.compare in ("merudra", "pufivik"):
-        alone = (merudra_kernels_alone if args.compare == "merudra" else pufivik_kernels_alone)(torch, ops, peaks)
+    alone_of = {"merudra": merudra_kernels_alone, "pufivik": pufivik_kernels_alone, "zugunex": zugunex_kernels_alone}
+    if not args.compare_size and args.compare in alone_of:
+        alone = alone_of[args.compare](torch, ops, peaks)
     clocks.stop()
     title = {"besavik": "Besavik beside Ganidra and Qwen3", "merudra": "Merudra beside Besavik and Qwen3",
              "pufivik": "Pufivik beside Merudra and Qwen3", "zugunex": "Zugunex beside Besavik and Qwen3"}.get(args.compare, "Ganidra beside Qwen3")

@@ -71,40 +71,6 @@ struct __align__(1024) PrSmem {
   int abort_flag;
 };
 
-// 32 rows x COLS bfloat16 columns of the output, from the warp whose lane l holds row l (as the accumulator leaves
-// tensor memory: packed[i] = columns 2 i, 2 i + 1 of the lane's row), to memory with lanes along the columns: through
-// 4 KB of shared memory of the warp's own (16-byte chunks XORed with the row's low bits), then 128 or 64 bytes of a
-// row per 8 or 4 lanes.  Stored with lanes along the rows, every instruction touched 32 rows with 16 bytes each, and a
-// tile's epilogue took 3.5-5.8 us (measured with the timeline build), as long as its products.
-// dst: row 0, column 0 of the 32 x COLS block; ld: elements per row of the output; rows, cols: how many of them exist.
-template <int COLS>
-__device__ __forceinline__ void pr_store_block(unsigned char* wst, const uint32_t (&packed)[COLS / 2], __nv_bfloat16* dst, size_t ld,
-                                               int rows, int cols, int lane) {
-  constexpr int CH = COLS / 8, RB = COLS * 2, RPI = 32 / CH;     // chunks per row, bytes per row, rows per instruction
-#pragma unroll
-  for (int j = 0; j < CH; ++j)
-    *reinterpret_cast<uint4*>(wst + lane * RB + ((j ^ (lane & (CH - 1))) << 4)) =
-        make_uint4(packed[4 * j], packed[4 * j + 1], packed[4 * j + 2], packed[4 * j + 3]);
-  __syncwarp();
-  const int cj = lane % CH;
-#pragma unroll
-  for (int i = 0; i < CH; ++i) {
-    const int rr = i * RPI + lane / CH;
-    const uint4 v = *reinterpret_cast<const uint4*>(wst + rr * RB + ((cj ^ (rr & (CH - 1))) << 4));
-    if (rr < rows) {
-      __nv_bfloat16* d = dst + (size_t)rr * ld + cj * 8;
-      if (cj * 8 + 8 <= cols) {
-        *reinterpret_cast<uint4*>(d) = v;
-      } else {
-        const __nv_bfloat16* e = reinterpret_cast<const __nv_bfloat16*>(&v);
-        for (int k = 0; k < 8; ++k)
-          if (cj * 8 + k < cols) d[k] = e[k];
-      }
-    }
-  }
-  __syncwarp();
-}
-
 // K split over S pairs of a cluster: CTA (pair `cpair`, parity `rank`) finishes 1 / S of the columns of its 128 rows.
 // `stg`: this CTA's sums in shared memory, row r at r x BN x 4 bytes, 16-byte chunks XORed with the row's low bits;
 // the other shares lie at the same place in the CTAs of the same parity.  The loads of four chunks' shares are all

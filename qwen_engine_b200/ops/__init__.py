@@ -773,7 +773,8 @@ class DeviceWaitTimeout(RuntimeError):
 
 
 _STATUS_WORDS = ("qe_gemm_tc", "qe_gemm_tc_swap", "qe_gemm_tc_pair", "qe_gemm_tc_splitk", "qe_flash_attention_tc",
-                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode", "qe_moe_tc", "qe_latent_attention_tc")
+                 "qe_flash_attention", "qe_decode_attention_mma", "qe_small_m", "qe_latent_decode", "qe_moe_tc", "qe_latent_attention_tc",
+                 "qe_head_linear_tc")
 
 
 def device_status() -> dict[str, int]:
@@ -1475,6 +1476,9 @@ def latent_prepare(down: Optional[torch.Tensor], q: torch.Tensor, norm_w: Option
            "latent_prepare")
 
 
+HEAD_LINEAR_TC_MIN_M = 65      # rows from which the products with one matrix per head run on tcgen05
+
+
 def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stride: int, out_head_stride: int,
                 gate: Optional[torch.Tensor] = None) -> None:
     """out[t, h * out_head_stride + n] = sum_k w[h, n, k] x[t, h * x_head_stride + k]: one matrix per head, w [H, N, K];
@@ -1490,6 +1494,13 @@ def head_linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stri
     if gate is not None:
         _rows(gate, "head_linear: gate")
         _need(gate.shape == (M, H) and gate.dtype == w.dtype, "head_linear: gate must be [T, H] in w's dtype")
+    if (TCGEN05_ENABLED and x.dtype == torch.bfloat16 and M >= HEAD_LINEAR_TC_MIN_M and K % 8 == 0
+            and not any(v % 8 for v in (x.stride(0), x_head_stride, out.stride(0), out_head_stride))
+            and x.data_ptr() % 16 == 0 and out.data_ptr() % 16 == 0):
+        _check(lib().qe_head_linear_tc(_ptr(x), ctypes.c_long(x.stride(0)), ctypes.c_long(x_head_stride), _ptr(w), _ptr(out),
+                                       ctypes.c_long(out.stride(0)), ctypes.c_long(out_head_stride), M, H, N, K, _ptr(gate),
+                                       ctypes.c_long(gate.stride(0) if gate is not None else 0), _stream()), "head_linear")
+        return
     _check(lib().qe_head_linear(_ptr(x), ctypes.c_long(x.stride(0)), ctypes.c_long(x_head_stride), _ptr(w), _ptr(out),
                                 ctypes.c_long(out.stride(0)), ctypes.c_long(out_head_stride), M, H, N, K, _dt(x), _ptr(gate),
                                 ctypes.c_long(gate.stride(0) if gate is not None else 0), _stream()), "head_linear")

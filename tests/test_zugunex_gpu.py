@@ -108,7 +108,8 @@ def test_a_layer_that_reads_anothers_cache_only_turns_its_queries(ops, dtype, H,
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("M,H,N,K", [(1, 3, 24, 8), (70, 2, 10, 6), (130, 8, 64, 32), (8, 16, 128, 192), (33, 5, 129, 65)])
+@pytest.mark.parametrize("M,H,N,K", [(1, 3, 24, 8), (70, 2, 10, 6), (130, 8, 64, 32), (8, 16, 128, 192), (33, 5, 129, 65), (300, 3, 200, 72),
+                                     (65, 16, 192, 128), (1000, 2, 256, 264), (129, 5, 40, 8), (2050, 16, 128, 192), (70, 4, 520, 64)])
 def test_a_product_per_head_with_a_gate_per_head(ops, dtype, M, H, N, K):
     g = torch.Generator().manual_seed(M + N)
     xs = K + (8 if K % 8 == 0 else 3)
@@ -120,6 +121,12 @@ def test_a_product_per_head_with_a_gate_per_head(ops, dtype, M, H, N, K):
     xh = torch.stack([x[:, h * xs:h * xs + K] for h in range(H)], dim=1).double()
     want = torch.einsum("mhk,hnk->mhn", xh, w.double()) * torch.sigmoid(wide.double()[:, 2:2 + H, None])
     _close(out.reshape(M, H, N), want, dtype, "gated heads")
+    # heads further apart in the output than they are wide: what lies between them stays as it was
+    apart = torch.full((M, H * (N + 8) + 8), 9.0, dtype=dtype, device=DEV)
+    ops.head_linear(x.to(DEV), w.to(DEV), apart[:, :H * (N + 8)], xs, N + 8)
+    got = apart[:, :H * (N + 8)].reshape(M, H, N + 8)
+    _close(got[:, :, :N], torch.einsum("mhk,hnk->mhn", xh, w.double()), dtype, "heads")
+    assert bool((got[:, :, N:] == 9.0).all()) and bool((apart[:, H * (N + 8):] == 9.0).all()) and ops.device_status() == {}
 
 
 # ---- attention over a latent cache with a window and a sink ----------------------------------------------------------------
