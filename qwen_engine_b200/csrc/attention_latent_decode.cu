@@ -124,7 +124,8 @@ latent_decode_kernel(LaArgs A) {
 #pragma unroll
       for (int cb = 0; cb < (DT + 127) / 128; ++cb) {
         const int c8 = cb * 16 + ch;
-        if (c8 < chunks) la_cp16(dst + row * (LD * 2) + c8 * 16, ok ? src + c8 * 8 : A.pages, ok);
+        const bool there = ok && c8 < chunks;        // (channels behind the row's own count as zeros)
+        if (c8 < DT / 8) la_cp16(dst + row * (LD * 2) + c8 * 16, there ? src + c8 * 8 : A.pages, there);
       }
     }
   };
@@ -144,10 +145,10 @@ latent_decode_kernel(LaArgs A) {
     if (!early[s] && gidx < n_groups) issue(gidx, s);
     cp_async_commit();                              // one commit per stage, issued or not: the waits below count them
   }
-  for (int e = tid; e < LA_ROWS * chunks; e += LA_THREADS) {
-    const int r = e / chunks, c8 = e - r * chunks;
+  for (int e = tid; e < LA_ROWS * (DT / 8); e += LA_THREADS) {
+    const int r = e / (DT / 8), c8 = e % (DT / 8);
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < nrows) {
+    if (r < nrows && c8 < chunks) {
       const int ti = (first_row + r) / H, h = (first_row + r) - ti * H;
       v = __ldcg(reinterpret_cast<const uint4*>(A.q + (size_t)(row0 + q0 + ti) * A.q_stride + (size_t)h * D) + c8);
     }
@@ -158,7 +159,6 @@ latent_decode_kernel(LaArgs A) {
   // ---- this warp's groups --------------------------------------------------------------------------------------
   const int g = lane >> 2, c = lane & 3;
   const int pos_lo = first_pos + (first_row + g) / H, pos_hi = first_pos + (first_row + g + 8) / H;
-  const int nks = D >> 4, nvd = v_pad >> 4;
   float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
   float o[DT / 8][4];
 #pragma unroll
@@ -175,14 +175,12 @@ latent_decode_kernel(LaArgs A) {
 #pragma unroll
       for (int j = 0; j < 2; ++j) s[i][j][0] = s[i][j][1] = s[i][j][2] = s[i][j][3] = 0.f;
 #pragma unroll
-    for (int ks = 0; ks < DT / 16; ++ks) {
-      if (ks < nks) {
-        uint32_t a[4], b[4];
-        ldsm_x4(a, sq + (lane & 15) * LD + ks * 16 + (lane >> 4) * 8);
-        ldsm_x4(b, tk + ((lane >> 4) * 8 + (lane & 7)) * LD + ks * 16 + ((lane >> 3) & 1) * 8);
-        fa_mma(s[ks & 1][0], a, b[0], b[1]);
-        fa_mma(s[ks & 1][1], a, b[2], b[3]);
-      }
+    for (int ks = 0; ks < DT / 16; ++ks) {           // (no condition on the row's own channels: the loads of many steps stay in flight)
+      uint32_t a[4], b[4];
+      ldsm_x4(a, sq + (lane & 15) * LD + ks * 16 + (lane >> 4) * 8);
+      ldsm_x4(b, tk + ((lane >> 4) * 8 + (lane & 7)) * LD + ks * 16 + ((lane >> 3) & 1) * 8);
+      fa_mma(s[ks & 1][0], a, b[0], b[1]);
+      fa_mma(s[ks & 1][1], a, b[2], b[3]);
     }
     float p[2][4];
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
@@ -222,17 +220,15 @@ latent_decode_kernel(LaArgs A) {
     uint32_t pa[4] = {pack_bf16(p[0][0], p[0][1]), pack_bf16(p[0][2], p[0][3]), pack_bf16(p[1][0], p[1][1]), pack_bf16(p[1][2], p[1][3])};
 #pragma unroll
     for (int dp = 0; dp < DT / 16; ++dp) {
-      if (dp < nvd) {
-        uint32_t b[4];
-        ldsm_x4_t(b, tk + (((lane >> 3) & 1) * 8 + (lane & 7)) * LD + dp * 16 + (lane >> 4) * 8);
+      uint32_t b[4];
+      ldsm_x4_t(b, tk + (((lane >> 3) & 1) * 8 + (lane & 7)) * LD + dp * 16 + (lane >> 4) * 8);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          o[2 * dp][e] *= e < 2 ? al_lo : al_hi;
-          o[2 * dp + 1][e] *= e < 2 ? al_lo : al_hi;
-        }
-        fa_mma(o[2 * dp], pa, b[0], b[1]);
-        fa_mma(o[2 * dp + 1], pa, b[2], b[3]);
+      for (int e = 0; e < 4; ++e) {
+        o[2 * dp][e] *= e < 2 ? al_lo : al_hi;
+        o[2 * dp + 1][e] *= e < 2 ? al_lo : al_hi;
       }
+      fa_mma(o[2 * dp], pa, b[0], b[1]);
+      fa_mma(o[2 * dp + 1], pa, b[2], b[3]);
     }
     __syncwarp();                                   // every lane is done with the stage before it is filled again
     const int nxt = gidx + LA_STAGES * LA_WARPS;
