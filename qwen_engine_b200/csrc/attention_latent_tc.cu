@@ -92,35 +92,41 @@ latent_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gr
   pdl_wait();
 
   if (warp == 0) {
-    if (lane == 0) {
-      mbar_expect_tx(&bars.q_full, (uint32_t)CB * LT_ROWS * 128u);
-      for (int cb = 0; cb < CB; ++cb) tma_load_2d(sq + (size_t)cb * LT_ROWS * 128, &map_q, &bars.q_full, cb * 64, (row0 + q0) * H);
-      const int* table = A.block_tables + (size_t)req * A.max_blocks;
-      const int box_rows = min(A.page_size, LT_BN);               // (a power of two, at least 8)
-      const int boxes = LT_BN / box_rows;
-      bool ok = true;
-      int j = 0;
-      for (; j < n_steps; ++j) {
-        const int s = j % SLOTS, round = j / SLOTS;
-        if (round > 0 && !mbar_wait(&bars.k_empty[s], (round - 1) & 1, abort_flag, 51, &g_lt_status)) { ok = false; break; }
-        mbar_expect_tx(&bars.k_full[s], slot_bytes);
-        for (int b = 0; b < boxes; ++b) {
-          const int key = kt0 + j * LT_BN + b * box_rows;
-          const int blk = key / A.page_size, y = key - blk * A.page_size;
-          int page = (key < kv_end && key + box_rows > kv_begin && blk < A.max_blocks) ? __ldg(table + blk) : -1;
-          if (page < 0) page = A.num_pages;                       // outside the tensor: zeros
-          for (int cb = 0; cb < CB; ++cb)
-            tma_load_3d(sk + (size_t)s * slot_bytes + ((size_t)cb * LT_BN + (size_t)b * box_rows) * 128, &map_kv, &bars.k_full[s],
-                        cb * 64, y, page);
-        }
-      }
-      if (!ok) {
-        // giving up: let the copies that are still in flight land before the CTA leaves (bounded)
-        for (uint32_t spin = 0; spin < TC_WAIT_LIMIT; ++spin) if (mbar_try_wait(&bars.q_full, 0)) break;
-        for (int i = j > SLOTS ? j - SLOTS : 0; i < j; ++i)
-          for (uint32_t spin = 0; spin < TC_WAIT_LIMIT; ++spin) if (mbar_try_wait(&bars.k_full[i % SLOTS], (i / SLOTS) & 1)) break;
-      }
+    // the whole warp issues the loads, a lane per box of a step (a page and 64 channels)
+    if (lane == 0) mbar_expect_tx(&bars.q_full, (uint32_t)CB * LT_ROWS * 128u);
+    __syncwarp();
+    if (lane < CB) tma_load_2d(sq + (size_t)lane * LT_ROWS * 128, &map_q, &bars.q_full, lane * 64, (row0 + q0) * H);
+    const int* table = A.block_tables + (size_t)req * A.max_blocks;
+    const int box_rows = min(A.page_size, LT_BN);                 // (a power of two, at least 8: at most 8 boxes of 4 blocks a step)
+    const int page_shift = __ffs(A.page_size) - 1;
+    const int b = lane / CB, cb = lane - b * CB;
+    const bool mine = b < LT_BN / box_rows;
+    auto page_of = [&](int j) {                                   // the page of this lane's box of step j
+      const int key = kt0 + j * LT_BN + b * box_rows, blk = key >> page_shift;
+      int page = (mine && j < n_steps && key < kv_end && key + box_rows > kv_begin && blk < A.max_blocks) ? __ldg(table + blk) : -1;
+      return page < 0 ? A.num_pages : page;                       // outside the tensor: zeros
+    };
+    bool ok = true;
+    int j = 0, page = page_of(0);
+    for (; j < n_steps; ++j) {
+      const int s = j % SLOTS, round = j / SLOTS;
+      const int next_page = page_of(j + 1);
+      if (round > 0) ok = __all_sync(0xffffffffu, mbar_wait(&bars.k_empty[s], (round - 1) & 1, abort_flag, 51, &g_lt_status));
+      if (!ok) break;
+      if (lane == 0) mbar_expect_tx(&bars.k_full[s], slot_bytes);
+      __syncwarp();
+      if (mine)
+        tma_load_3d(sk + (size_t)s * slot_bytes + ((size_t)cb * LT_BN + (size_t)b * box_rows) * 128, &map_kv, &bars.k_full[s],
+                    cb * 64, (kt0 + j * LT_BN + b * box_rows) & (A.page_size - 1), page);
+      page = next_page;
     }
+    if (!ok && lane == 0) {
+      // giving up: let the copies that are still in flight land before the CTA leaves (bounded)
+      for (uint32_t spin = 0; spin < TC_WAIT_LIMIT; ++spin) if (mbar_try_wait(&bars.q_full, 0)) break;
+      for (int i = j > SLOTS ? j - SLOTS : 0; i < j; ++i)
+        for (uint32_t spin = 0; spin < TC_WAIT_LIMIT; ++spin) if (mbar_try_wait(&bars.k_full[i % SLOTS], (i / SLOTS) & 1)) break;
+    }
+    __syncwarp();
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = make_idesc(LT_ROWS, LT_BN);

@@ -38,7 +38,7 @@ import torch
 from .. import ops
 from ..cache.spec import PagedKVSpec
 from ..weights.spec import MATRIX, NORM, VECTOR, WeightSpec
-from .base import Mixer, StepContext, register
+from .base import Mixer, StepContext, register, step_hint
 
 _NAMES = dict(q="q", q_down="dq", q_norm="dq.norm", q_up="uq", kv_down="dkv", kv_norm="dkv.norm", k_up="uk", v_up="uv",
               gate="g", out="o", sink="sink")
@@ -195,5 +195,9 @@ class LatentAttention(Mixer):
 
     def forward(self, ctx: StepContext, x, cache, group, out, write_cache: bool = True) -> None:
         inner = ctx.arena.alloc((ctx.num_tokens, self.inner_width), ctx.dtype)
+        if self.query_rank is None:
+            ops.prefetch_next(self.w_o)              # (the product of a few rows asks L2 for the matrix the mixer ends with)
         self.mix_into(ctx, x, cache, group, inner, write_cache)
+        ops.prefetch_next(step_hint(ctx, "weights_after_mixer"))
         ops.linear(inner, self.w_o, out)
+        ops.prefetch_next(None)

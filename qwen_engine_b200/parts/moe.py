@@ -118,7 +118,8 @@ class RoutedExperts(FeedForward):
             self.correction = source.get(prefix + self.correction_name).to(torch.float32).to(device).contiguous()
 
     def first_weights(self):
-        return None
+        # (asked for ahead of time by a product of a few rows, where most experts are used and they fit on the chip)
+        return self.w_gate_up if not self.gated and self.num_experts <= 4 * self.top else None
 
     def forward(self, ctx: StepContext, x, out) -> None:
         T = ctx.num_tokens
