@@ -26,7 +26,7 @@
 #define MOE_MAX_TOP 32
 
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(512)
 moe_route_kernel(const T* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias,
                  int* __restrict__ top_idx, float* __restrict__ top_w, int T_tokens, int W, int E, int top, int scoring,
                  const float* __restrict__ correction, float weight_scale, int n_always) {
@@ -158,7 +158,9 @@ extern "C" int qe_moe_route(const void* x, const float* w, const float* bias, in
     if (e != cudaSuccess) QE_REFUSE("moe_route: shared memory: %s", cudaGetErrorString(e));
     configured = true;
   }
-#define MR(TT) qe_launch(moe_route_kernel<TT>, dim3(T), dim3(128), smem, stream, (const TT*)x, w, bias, top_idx, top_w, T, W, E, top, scoring, correction, weight_scale, n_always)
+  // a few tokens: more warps a token, so that its experts are scored at once (an expert's warp is the same code)
+  const int threads = T <= 148 && E > 4 ? (E > 8 ? 512 : 288) : 128;
+#define MR(TT) qe_launch(moe_route_kernel<TT>, dim3(T), dim3(threads), smem, stream, (const TT*)x, w, bias, top_idx, top_w, T, W, E, top, scoring, correction, weight_scale, n_always)
   if (dtype == QE_DTYPE_F32) MR(float);
   else if (dtype == QE_DTYPE_BF16) MR(__nv_bfloat16);
   else QE_REFUSE("moe_route: unknown dtype %d", dtype);
