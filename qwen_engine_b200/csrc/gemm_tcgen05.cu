@@ -41,7 +41,7 @@ struct __align__(1024) TcSmem {
 // STARVED (the self-test of the give-up path, qe_gemm_tc_selftest_starved): the producer issues no load and arms
 // no barrier, and the waits give up after `starved_limit` polls instead of TC_WAIT_LIMIT; everything else is
 // the product kernel as it is.
-template <typename TOut, int BN, int STAGES, bool STARVED = false>
+template <typename TOut, int BN, int STAGES, bool STARVED = false, bool ACT = false>
 __global__ void __launch_bounds__(TC_THREADS, 1)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                     TOut* __restrict__ out, int M, int N, int K, int starved_limit, int act) {
@@ -168,7 +168,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
           __syncwarp();
           if (lane == 0) mbar_arrive(&sm.acc_empty[buf]);
         }
-        if (act) {
+        if constexpr (ACT) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(act_for<TOut>(__uint_as_float(r[j]), act));
         }
@@ -232,24 +232,24 @@ extern "C" void qe_gemm_tc_clear_status() {
   cudaMemcpyToSymbol(g_tc_status, &v, sizeof(int));
 }
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool ACT>
 static int launch_tc(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, int sms, cudaStream_t stream, int act) {
   CUtensorMap map_x, map_w;
   if (!get_map(x, M, K, TC_BM, &map_x) || !get_map(w, N, K, BN, &map_w)) return 1;
   const size_t smem = sizeof(TcSmem<BN, STAGES>) + 1024;
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tcgen05_kernel<float, BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES, false, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tcgen05_kernel<float, BN, STAGES, false, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) QE_REFUSE("linear_tcgen05: shared memory %zu: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
   const long tiles = (long)((N + BN - 1) / BN) * ((M + TC_BM - 1) / TC_BM);
   const dim3 grid((unsigned)(tiles < sms ? tiles : sms));
   if (out_f32)
-    qe_launch(gemm_tcgen05_kernel<float, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (float*)out, M, N, K, 0, act);
+    qe_launch(gemm_tcgen05_kernel<float, BN, STAGES, false, ACT>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (float*)out, M, N, K, 0, act);
   else
-    qe_launch(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (__nv_bfloat16*)out, M, N, K, 0, act);
+    qe_launch(gemm_tcgen05_kernel<__nv_bfloat16, BN, STAGES, false, ACT>, grid, dim3(TC_THREADS), smem, stream, map_x, map_w, (__nv_bfloat16*)out, M, N, K, 0, act);
   QE_CHECK_LAUNCH("linear_tcgen05");
   return 0;
 }
@@ -296,6 +296,8 @@ extern "C" int qe_linear_tcgen05(const void* x, const void* w, void* out, int M,
   const int sms = sm_count();
   // wide tiles reuse the fetched rows of x twice as often; narrow ones when wide ones would leave SMs idle
   const long wide_tiles = (long)((N + 255) / 256) * ((M + TC_BM - 1) / TC_BM);
-  if (wide_tiles >= sms) return launch_tc<256, 4>(x, w, out, M, N, K, out_f32, sms, stream, act);
-  return launch_tc<128, 6>(x, w, out, M, N, K, out_f32, sms, stream, act);
+#define TC_GO(ACT) (wide_tiles >= sms ? launch_tc<256, 4, ACT>(x, w, out, M, N, K, out_f32, sms, stream, act) \
+                                      : launch_tc<128, 6, ACT>(x, w, out, M, N, K, out_f32, sms, stream, act))
+  return act ? TC_GO(true) : TC_GO(false);
+#undef TC_GO
 }

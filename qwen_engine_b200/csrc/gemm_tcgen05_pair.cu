@@ -75,7 +75,7 @@ struct __align__(1024) PrSmem {
 // `stg`: this CTA's sums in shared memory, row r at r x BN x 4 bytes, 16-byte chunks XORed with the row's low bits;
 // the other shares lie at the same place in the CTAs of the same parity.  The loads of four chunks' shares are all
 // in flight before the first is used (a load from another CTA's shared memory takes some hundreds of cycles).
-template <typename TOut, int BN, int S>
+template <typename TOut, int BN, int S, bool ACT>
 __device__ __forceinline__ void pr_meet_shares(const unsigned char* stg, TOut* __restrict__ out, int M, int N, int m0, int n0,
                                                uint32_t rank, uint32_t cpair, int act) {
   constexpr int CPR = (BN / 4) / S;                  // 16-byte chunks of a row that this CTA finishes
@@ -103,7 +103,7 @@ __device__ __forceinline__ void pr_meet_shares(const unsigned char* stg, TOut* _
       float4 acc = v[b][0];                          // in the order of the shares
 #pragma unroll
       for (int sp = 1; sp < S; ++sp) { acc.x += v[b][sp].x; acc.y += v[b][sp].y; acc.z += v[b][sp].z; acc.w += v[b][sp].w; }
-      if (act) {
+      if constexpr (ACT) {
         acc.x = act_for<TOut>(acc.x, act); acc.y = act_for<TOut>(acc.y, act);
         acc.z = act_for<TOut>(acc.z, act); acc.w = act_for<TOut>(acc.w, act);
       }
@@ -121,7 +121,8 @@ __device__ __forceinline__ void pr_meet_shares(const unsigned char* stg, TOut* _
 }
 
 // N: columns of the product (SWIGLU: 2 I); n_up: SWIGLU: the first row of up in w (= I), else 0
-template <typename TOut, int BN, int STAGES, bool SWIGLU, bool ROPE = false>
+// ACT: a plain product whose sums pass the activation gate_act (common.cuh: act_for)
+template <typename TOut, int BN, int STAGES, bool SWIGLU, bool ROPE = false, bool ACT = false>
 __global__ void __launch_bounds__(PR_THREADS, 1)
 gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
                          TOut* __restrict__ out, int M, int N, int K, int n_up, PrRope rp, int splits, int gate_act) {
@@ -468,7 +469,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
         tc_fence_before();
         __syncwarp();
         if (lane == 0) mbar_arrive_cluster(smem_u32(&sm.acc_empty[buf]) & TC_PEER_BIT_MASK);
-        if (gate_act) {                              // (a plain product: the activation of its sums)
+        if constexpr (ACT) {
 #pragma unroll
           for (int q = 0; q < NLD; ++q)
 #pragma unroll
@@ -502,7 +503,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
           __syncwarp();
           if (lane == 0) mbar_arrive_cluster(smem_u32(&sm.acc_empty[buf]) & TC_PEER_BIT_MASK);
         }
-        if (gate_act) {
+        if constexpr (ACT) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(act_for<TOut>(__uint_as_float(r[j]), gate_act));
         }
@@ -536,8 +537,8 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
     if (warp >= 2 && split_staged) {
       const int tile = pair;
       const int m0 = (tile / n_blocks) * 2 * PR_BM + (int)rank * PR_BM, n0 = (tile % n_blocks) * BN;
-      if (splits == 2) pr_meet_shares<TOut, BN, 2>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
-      else pr_meet_shares<TOut, BN, 4>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
+      if (splits == 2) pr_meet_shares<TOut, BN, 2, ACT>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
+      else pr_meet_shares<TOut, BN, 4, ACT>(reinterpret_cast<const unsigned char*>(sm.a), out, M, N, m0, n0, rank, cpair, gate_act);
     }
   }
   // both CTAs meet here: neither leaves while the other may still signal its barriers, read its
@@ -554,7 +555,7 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
   QE_TL_FLUSH_STAMPS();
 }
 
-template <int BN, int STAGES, bool SWIGLU = false, bool ROPE = false>
+template <int BN, int STAGES, bool SWIGLU = false, bool ROPE = false, bool ACT = false>
 static int launch_pair(const void* x, const void* w, void* out, int M, int N, int K, int out_f32, int sms, cudaStream_t stream,
                        PrRope rp = PrRope{}, int splits = 1, int gate_act = 0) {
   const int n_up = SWIGLU ? N / 2 : 0;
@@ -580,9 +581,9 @@ static int launch_pair(const void* x, const void* w, void* out, int M, int N, in
 #endif
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<__nv_bfloat16, BN, STAGES, SWIGLU, ROPE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<__nv_bfloat16, BN, STAGES, SWIGLU, ROPE, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if constexpr (!ROPE)
-      if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<float, BN, STAGES, SWIGLU, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+      if (e == cudaSuccess) e = cudaFuncSetAttribute(gemm_tcgen05_pair_kernel<float, BN, STAGES, SWIGLU, false, ACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) QE_REFUSE("linear_tcgen05_pair: shared memory %zu: %s", smem, cudaGetErrorString(e));
     configured = true;
   }
@@ -596,9 +597,9 @@ static int launch_pair(const void* x, const void* w, void* out, int M, int N, in
     qe_launch_cluster(gemm_tcgen05_pair_kernel<__nv_bfloat16, BN, STAGES, false, true>, grid, dim3(PR_THREADS), smem, stream, cluster, map_x, map_w, (__nv_bfloat16*)out, M, N, K, n_up, rp, 1, 0);
   } else {
     if (out_f32)
-      qe_launch_cluster(gemm_tcgen05_pair_kernel<float, BN, STAGES, SWIGLU, false>, grid, dim3(PR_THREADS), smem, stream, cluster, map_x, map_w, (float*)out, M, N, K, n_up, rp, splits, gate_act);
+      qe_launch_cluster(gemm_tcgen05_pair_kernel<float, BN, STAGES, SWIGLU, false, ACT>, grid, dim3(PR_THREADS), smem, stream, cluster, map_x, map_w, (float*)out, M, N, K, n_up, rp, splits, gate_act);
     else
-      qe_launch_cluster(gemm_tcgen05_pair_kernel<__nv_bfloat16, BN, STAGES, SWIGLU, false>, grid, dim3(PR_THREADS), smem, stream, cluster, map_x, map_w, (__nv_bfloat16*)out, M, N, K, n_up, rp, splits, gate_act);
+      qe_launch_cluster(gemm_tcgen05_pair_kernel<__nv_bfloat16, BN, STAGES, SWIGLU, false, ACT>, grid, dim3(PR_THREADS), smem, stream, cluster, map_x, map_w, (__nv_bfloat16*)out, M, N, K, n_up, rp, splits, gate_act);
   }
   QE_CHECK_LAUNCH("linear_tcgen05_pair");
   return 0;
@@ -699,9 +700,11 @@ extern "C" int qe_linear_tcgen05_pair(const void* x, const void* w, void* out, i
   if (sms < 2) QE_REFUSE("linear_tcgen05_pair: needs at least two SMs");
   // wide tiles, wide tiles with K split over 2 or 4 pairs, or narrow tiles: see qe_tc_product_plan
   const int plan = qe_tc_product_plan(M, N, K, 1);
-  if (plan == 2) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, 1, act);
-  if (plan >= 3) return launch_pair<256, 6>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, plan == 3 ? 2 : 4, act);
-  return launch_pair<128, 8>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, 1, act);
+  const int splits = plan == 3 ? 2 : plan == 4 ? 4 : 1;
+#define PR_GO(ACT) (plan >= 2 ? launch_pair<256, 6, false, false, ACT>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, splits, act) \
+                              : launch_pair<128, 8, false, false, ACT>(x, w, out, M, N, K, out_f32, sms, stream, PrRope{}, 1, act))
+  return act ? PR_GO(true) : PR_GO(false);
+#undef PR_GO
 }
 
 // out[M, I] = silu(x · w[:I]^T) * (x · w[I:]^T) for the stacked gate and up weights w [2 I, K] (see SWIGLU
