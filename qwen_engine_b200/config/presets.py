@@ -117,6 +117,20 @@ PRESETS: dict[str, dict[str, Any]] = {
                                             rot=dict(base=20000.0, dims=16), kv_from=0),
                                  mlp=None)]),
         init=dict(seed=23, std=0.08, norm_std=0.1, block_size=16)),
+    # a small model of the Funudra design: state-space layers, and softmax attention (bent scores, convolutions of q, k and
+    # v, values larger than keys) beside a matrix memory; the last layer is the first one's weights once more
+    "funudra-tiny": dict(
+        config=dict(architecture="Funudra", vocab=320, width=128, norm=dict(eps=1e-6),
+                    layers=[dict(type="mamba2", mixer=dict(heads=4, vdim=32, state=32, groups=2, conv=4, norm_groups=2),
+                                 mlp=dict(kind="dense", ff=256)),
+                            dict(type="parallel",
+                                 mixer=dict(left=dict(heads=4, kv_heads=2, dim=32, vdim=48, conv=3, scale=0.2, softcap=20.0,
+                                                      rot=dict(base=10000.0, dims=16, scaling=dict(factor=4.0))),
+                                            right=dict(heads=2, dim=32, vdim=40, gate_cap=8.0), left_scale=0.7, right_scale=0.4),
+                                 mlp=dict(kind="dense", ff=192)),
+                            dict(type="mamba2", mixer=dict(heads=4, vdim=32, state=32, groups=2, conv=4, norm_groups=2),
+                                 mlp=dict(kind="dense", ff=256), weights_of=0)]),
+        init=dict(seed=29, std=0.08, norm_std=0.1, block_size=16)),
 }
 
 

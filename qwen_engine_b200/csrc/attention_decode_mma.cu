@@ -105,9 +105,9 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
 
   const int* __restrict__ table = A.block_tables + (size_t)req * A.max_blocks;
   const int page_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
-  const size_t page_stride = (size_t)(A.kv_planes == 1 ? 1 : 2) * Hkv * page_size * D;
+  const size_t page_stride = (size_t)A.kv_planes * Hkv * page_size * D;
   // (the values of kv head (hkv + v_shift) mod Hkv where the weights of this one are to meet another's)
-  const size_t v_off = A.kv_planes == 1 ? 0 : ((size_t)Hkv + (size_t)((hkv + A.v_shift) % Hkv) - (size_t)hkv) * page_size * D;
+  const size_t v_off = A.kv_planes == 1 ? 0 : ((size_t)Hkv * (1 + A.v_plane) + (size_t)((hkv + A.v_shift) % Hkv) - (size_t)hkv) * page_size * D;
   const __nv_bfloat16* head_base = A.pages + (size_t)hkv * page_size * D;
   // a group that starts at a multiple of 16 keys lies in one page when pages are multiples of 16 keys
   const bool one_page = page_shift >= 4 && (kv_begin & 15) == 0;
@@ -250,7 +250,8 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
   }
   __syncthreads();
   float* fin = reinterpret_cast<float*>(stages) + DM_ROWS * D;        // CL: [16][128] after warp 0's result
-  __nv_bfloat16* out_row0 = A.out + (size_t)(row0 + q0) * ((size_t)Hq * D);
+  const int out_hd = A.out_hd;
+  __nv_bfloat16* out_row0 = A.out + (size_t)(row0 + q0) * ((size_t)Hq * out_hd);
   for (int e = tid; e < nrows * D; e += DM_THREADS) {
     const int r = e / D, d = e - r * D;
     float m = -INFINITY;
@@ -270,7 +271,7 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
     } else if (part < 0) {
       const int ti = r / G, hg = r - ti * G;
       if (A.sinks) l += exp2f(A.sinks[hkv * G + hg] * 1.4426950408889634f - mb);      // the sink's share of the denominator
-      out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+      out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
     } else {
       const size_t slot = ((size_t)part * Hkv + hkv) * A.part_rows + r;
       A.part_acc[slot * D + d] = acc;
@@ -340,7 +341,7 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
         }
         const int ti = r / G, hg = r - ti * G;
         if (A.sinks) l += exp2f(A.sinks[hkv * G + hg] * 1.4426950408889634f - mb);    // the sink's share of the denominator
-        out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+        out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
       }
       return;
     }
@@ -376,7 +377,7 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
         }
         const int ti = r / G, hg = r - ti * G;
         if (A.sinks) l += exp2f(A.sinks[hkv * G + hg] * 1.4426950408889634f - mb);    // the sink's share of the denominator
-        out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+        out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
       }
     }
     cluster_sync_all();                             // nobody reads this CTA's shared memory any more
@@ -410,7 +411,7 @@ decode_attention_mma_kernel(FaArgs A_launch, long long prefetch_delta, int early
         }
         const int ti = r / G, hg = r - ti * G;
         if (A.sinks) l += exp2f(A.sinks[hkv * G + hg] * 1.4426950408889634f - mb);    // the sink's share of the denominator
-        out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+        out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
       }
     }
   }
@@ -479,8 +480,9 @@ extern "C" int qe_decode_attention_mma(const void* q, long q_stride, const void*
                                        float softcap, const float* sinks, int v_shift, int shifts, long shift_out_stride,
                                        int shift_parts, cudaStream_t stream) {
   if (n_items <= 0) return 0;
-  if (shifts < 1 || shifts > Hkv || (shifts > 1 && kv_planes == 1)) QE_REFUSE("decode_attention_mma: %d shifts in one launch over %d kv heads", shifts, Hkv);
-  if (v_shift < 0 || v_shift >= Hkv || (v_shift && kv_planes == 1)) QE_REFUSE("decode_attention_mma: a shift of %d over %d kv heads", v_shift, Hkv);
+  if (kv_planes > 2 ? shifts != kv_planes - 1 : (shifts < 1 || shifts > Hkv || (shifts > 1 && kv_planes == 1)))
+    QE_REFUSE("decode_attention_mma: %d shifts in one launch over %d kv heads and %d planes", shifts, Hkv, kv_planes);
+  if (kv_planes < 1 || v_shift < 0 || v_shift >= Hkv || (v_shift && kv_planes != 2)) QE_REFUSE("decode_attention_mma: a shift of %d over %d kv heads", v_shift, Hkv);
   if (slopes && softcap > 0.f) QE_REFUSE("decode_attention_mma: scores are biased by distance or bent, not both");
   if (!qe_decode_attention_mma_supported(Hq, Hkv, D, max_rows))
     QE_REFUSE("decode_attention_mma: heads %d/%d, head_dim %d, %d rows are not supported", Hq, Hkv, D, max_rows);
@@ -490,7 +492,8 @@ extern "C" int qe_decode_attention_mma(const void* q, long q_stride, const void*
   if (part_acc && counters == nullptr && !cluster) QE_REFUSE("decode_attention_mma: parts need the counters");
   FaArgs fa{(const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)pages, block_tables, max_blocks, items,
             (__nv_bfloat16*)out, part_acc, part_ml, part_rows, counters, scale * 1.4426950408889634f, window, Hq, Hkv,
-            page_size, slopes, kv_planes, softcap, scale, sinks, v_shift, shift_out_stride, shift_parts};
+            page_size, slopes, kv_planes, softcap, scale, sinks, v_shift, shift_out_stride, shift_parts,
+            DM_D * (kv_planes > 2 ? kv_planes - 1 : 1), 0};
   if (cluster == 0) return launch_decode_mma<false>(fa, delta, n_items, Hkv, 0, wide, max_rows, stream, shifts);
   if ((cluster != 2 && cluster != 4 && cluster != 8) || n_items % cluster)
     QE_REFUSE("decode_attention_mma: %d items cannot form clusters of %d", n_items, cluster);

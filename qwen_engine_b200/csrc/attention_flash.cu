@@ -67,7 +67,7 @@ static int launch_flash(const void* q, long q_stride, const void* pages, const i
   dim3 grid(n_items, Hkv, shifts);
   FaArgs fa{(const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)pages, block_tables, max_blocks, items,
             (__nv_bfloat16*)out, part_acc, part_ml, part_rows, counters, scale_log2, window, Hq, Hkv, page_size, slopes, kv_planes,
-            softcap, scale, sinks, v_shift, shift_out_stride, shift_parts};
+            softcap, scale, sinks, v_shift, shift_out_stride, shift_parts, D * (kv_planes > 2 ? kv_planes - 1 : 1), 0};
   qe_launch(flash_attention_kernel<D, STAGES, QROWS>, grid, dim3(2 * FA_THREADS), smem, stream, fa);
   QE_CHECK_LAUNCH("flash_attention");
   if (n_merge > 0 && counters == nullptr) {
@@ -130,9 +130,11 @@ extern "C" int qe_flash_attention_fused_merge(const void* q, long q_stride, cons
   if (!qe_flash_attention_supported(Hq, Hkv, D))
     QE_REFUSE("flash_attention: heads %d/%d with head_dim %d are not supported", Hq, Hkv, D);
   if (((uintptr_t)q | (uintptr_t)pages) & 15 || (q_stride % 8)) QE_REFUSE("flash_attention: operands must be 16-byte aligned");
-  if (v_shift < 0 || v_shift >= Hkv || (v_shift && kv_planes == 1)) QE_REFUSE("flash_attention: a shift of %d over %d kv heads", v_shift, Hkv);
+  if (kv_planes < 1 || v_shift < 0 || v_shift >= Hkv || (v_shift && kv_planes != 2)) QE_REFUSE("flash_attention: a shift of %d over %d kv heads", v_shift, Hkv);
   // several shifts in one launch: each has its own output, parts and counters; the merge kernel is not laid out for them
-  if (shifts < 1 || shifts > Hkv || (shifts > 1 && (kv_planes == 1 || (n_merge > 0 && counters == nullptr))))
+  // (with more than two planes: the blocks of values)
+  if (kv_planes > 2 ? (shifts != kv_planes - 1 || (n_merge > 0 && counters == nullptr))
+                    : (shifts < 1 || shifts > Hkv || (shifts > 1 && (kv_planes == 1 || (n_merge > 0 && counters == nullptr)))))
     QE_REFUSE("flash_attention: %d shifts in one launch over %d kv heads", shifts, Hkv);
   if (slopes && softcap > 0.f) QE_REFUSE("flash_attention: scores are biased by distance or bent, not both");
 #define FA_ARGS q, q_stride, pages, block_tables, max_blocks, cu_q, ctx_lens, items, n_items, merge_items, n_merge, out, \

@@ -191,7 +191,7 @@ template <int D>
 __device__ __forceinline__ void fa_merge_parts(const float* part_acc, const float* part_ml, int part_rows, int first,
                                                int n, int hkv, int Hkv, int nrows, int G, int Hq,
                                                __nv_bfloat16* out_row0 /* row of the tile's first token */,
-                                               const float* sinks = nullptr) {
+                                               const float* sinks = nullptr, int out_hd = D) {
   for (int e = threadIdx.x; e < nrows * D; e += FA_THREADS) {       // the computing threads only
     const int r = e / D, d = e - r * D;
     float m = -INFINITY;
@@ -206,7 +206,7 @@ __device__ __forceinline__ void fa_merge_parts(const float* part_acc, const floa
     }
     const int ti = r / G, hg = r - ti * G;
     if (sinks) l += exp2f(sinks[hkv * G + hg] * 1.4426950408889634f - m);      // the sink's share of the denominator
-    out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+    out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
   }
 }
 
@@ -276,7 +276,8 @@ struct FaArgs {
   float* part_acc; float* part_ml; int part_rows;
   int* counters; float scale_log2; int window, Hq, Hkv, page_size;
   const float* slopes;      // null, or float32 [Hq]: slopes[h] * (position - key) is taken off the score (last: may be left out)
-  int kv_planes;            // 1: a page holds one plane per kv head and the values are its channels (a latent cache); else keys and values apart
+  int kv_planes;            // planes of a page: 1, the values are the keys' channels (a latent cache); 2, keys and values; 1 + n, keys and n
+                            // blocks of D value channels (values of n D channels): block v_plane is the one this launch works on
   float softcap;            // above 0: the scaled score s becomes softcap * tanh(s / softcap)
   float scale;              // the scale itself (scale_log2 / log2 e), for the bent scores
   const float* sinks;       // null, or float32 [Hq]: exp(sinks[h]) joins head h's denominator (no key, no value)
@@ -285,12 +286,15 @@ struct FaArgs {
   // output, of the parts' scratch and of the counters (fa_for_shift moves the pointers, so nothing else sees it).
   long shift_out_stride;    // elements between the outputs of two shifts
   int shift_parts;          // parts of one shift (their scratch and counters are laid out shift after shift)
+  int out_hd;               // elements between a token's heads in `out` (D; n D where a head has n blocks of values)
+  int v_plane;              // the block of values (with more than two planes the z dimension runs over the blocks, not over shifts)
 };
 
 __device__ __forceinline__ FaArgs fa_for_shift(const FaArgs& in, int z, int head_dim) {
   FaArgs A = in;
   if (z > 0) {
-    A.v_shift = (in.v_shift + z) % in.Hkv;
+    if (in.kv_planes > 2) A.v_plane = z;
+    else A.v_shift = (in.v_shift + z) % in.Hkv;
     A.out = in.out + (size_t)z * in.shift_out_stride;
     const size_t slots = (size_t)z * in.shift_parts * in.Hkv * in.part_rows;
     if (in.part_acc) A.part_acc = in.part_acc + slots * head_dim;
@@ -372,8 +376,8 @@ __device__ __forceinline__ void flash_attention_cta(const FaArgs& A, int item_id
     const int* table = block_tables + (size_t)req * max_blocks;
     // address arithmetic of the gather, hoisted: a page's stride, this head's offset in a page, K -> V
     const int page_shift = (page_size & (page_size - 1)) == 0 ? __ffs(page_size) - 1 : -1;
-    const size_t page_stride = (size_t)(A.kv_planes == 1 ? 1 : 2) * Hkv * page_size * D;
-    const size_t v_off = A.kv_planes == 1 ? 0 : (size_t)Hkv * page_size * D;
+    const size_t page_stride = (size_t)A.kv_planes * Hkv * page_size * D;
+    const size_t v_off = A.kv_planes == 1 ? 0 : (size_t)(1 + A.v_plane) * Hkv * page_size * D;
     const __nv_bfloat16* head_base = pages + (size_t)hkv * page_size * D;
     const long v_head_off = ((long)((hkv + A.v_shift) % Hkv) - hkv) * page_size * D;     // values of another kv head (0: its own)
     bool waited = false;
@@ -480,7 +484,8 @@ __device__ __forceinline__ void flash_attention_cta(const FaArgs& A, int item_id
     if (lane == 0) fa_bar_arrive(&bar_empty[stage]);      // this warp is done with the slot
   }
   if (ok) {                                         // else a wait ran out: the status flag says so; nothing is written
-  __nv_bfloat16* out_row0 = out + (size_t)(row0 + q0) * ((size_t)Hq * D);
+  const int out_hd = A.out_hd;
+  __nv_bfloat16* out_row0 = out + (size_t)(row0 + q0) * ((size_t)Hq * out_hd);
   if (keysplit) {
     // ---- combine the four warps' shares of the keys in shared memory (the tiles are done) ------
     fa_consumer_sync();
@@ -512,7 +517,7 @@ __device__ __forceinline__ void flash_attention_cta(const FaArgs& A, int item_id
       if (part < 0) {
         const int ti = r / G, hg = r - ti * G;
         if (sinks) l += exp2f(sinks[hkv * G + hg] * 1.4426950408889634f - base);
-        out_row0[(size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
+        out_row0[(size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd + d] = __float2bfloat16_rn(l > 0.f ? acc / l : 0.f);
       } else {
         const size_t slot = ((size_t)part * Hkv + hkv) * part_rows + r;
         part_acc[slot * D + d] = acc;
@@ -529,7 +534,7 @@ __device__ __forceinline__ void flash_attention_cta(const FaArgs& A, int item_id
       const float l = half ? l_hi : l_lo, m = half ? m_hi : m_lo;
       if (part < 0) {
         const float inv = 1.f / (sinks ? l + exp2f(sinks[hkv * G + hg] * 1.4426950408889634f - m) : l);
-        __nv_bfloat16* dst = out_row0 + (size_t)ti * ((size_t)Hq * D) + (size_t)(hkv * G + hg) * D;
+        __nv_bfloat16* dst = out_row0 + (size_t)ti * ((size_t)Hq * out_hd) + (size_t)(hkv * G + hg) * out_hd;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i) {
           const float v0 = o[i][2 * half] * inv, v1 = o[i][2 * half + 1] * inv;
@@ -559,7 +564,7 @@ __device__ __forceinline__ void flash_attention_cta(const FaArgs& A, int item_id
     fa_consumer_sync();
     if (s_last) {
       __threadfence();
-      fa_merge_parts<D>(part_acc, part_ml, part_rows, first, n_splits, hkv, Hkv, nrows, G, Hq, out_row0, sinks);
+      fa_merge_parts<D>(part_acc, part_ml, part_rows, first, n_splits, hkv, Hkv, nrows, G, Hq, out_row0, sinks, out_hd);
     }
   }
   }   // ok

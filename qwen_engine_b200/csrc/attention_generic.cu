@@ -12,7 +12,8 @@
 //
 // Options of other designs: `softcap` > 0 bends the scaled score s to softcap tanh(s / softcap) ahead of the mask; `sinks`
 // [Hq] adds exp(sinks[h]) to head h's denominator (no key, no value); `v_shift` lets a head whose kv head is c read the
-// values of kv head (c + v_shift) mod Hkv (the keys stay its own).
+// values of kv head (c + v_shift) mod Hkv (the keys stay its own).  A page of 1 + n planes (n > 1) holds the keys and n blocks of
+// D value channels; the grid's z runs over the blocks and a head's output has n D channels.
 //
 // One CTA per (tile of 16 queries of one request, query head); 4 warps, 4 queries each.  Within a
 // warp lane j owns key j of the tile for the scores and dims d = lane + 32 i of the output.
@@ -81,7 +82,7 @@ attention_generic_kernel(const T* __restrict__ q, long q_stride, const T* __rest
         // (kv_planes 1: a page holds one plane per kv head, and the values are its channels)
         const size_t base = ((((size_t)page * kv_planes) * Hkv + hkv) * page_size + (kj % page_size)) * D + d;
         kvl = to_f32(pages[base]);
-        vvl = kv_planes == 1 ? kvl : to_f32(pages[base + ((size_t)Hkv + hv - hkv) * page_size * D]);
+        vvl = kv_planes == 1 ? kvl : to_f32(pages[base + ((size_t)Hkv * (1 + blockIdx.z) + hv - hkv) * page_size * D]);
       }
       ks[j * Dp + d] = kvl;
       vs[j * D + d] = vvl;
@@ -126,7 +127,7 @@ attention_generic_kernel(const T* __restrict__ q, long q_stride, const T* __rest
     if (r >= nq) continue;
     // a sink: exp(sinks[head]) joins the denominator; it has no key and no value
     const float inv = 1.f / (sinks ? l[i] + expf(sinks[hq] - m[i]) : l[i]);
-    T* o = out + (size_t)(row0 + q0 + r) * ((size_t)Hq * D) + (size_t)hq * D;
+    T* o = out + (((size_t)(row0 + q0 + r) * Hq + hq) * gridDim.z + blockIdx.z) * D;
 #pragma unroll
     for (int c = 0; c < DREG; ++c) {
       const int d = lane + 32 * c;
@@ -146,7 +147,7 @@ extern "C" int qe_paged_attention_generic(const void* q, long q_stride, const vo
   if (Hkv < 1 || Hq % Hkv) QE_REFUSE("paged_attention: %d query heads do not group over %d kv heads", Hq, Hkv);
   if (Hq > 65535) QE_REFUSE("paged_attention: too many heads (%d)", Hq);
   const size_t smem = ((size_t)AG_BM * D + (size_t)AG_BN * (D + 1) + (size_t)AG_BN * D) * sizeof(float);
-  dim3 grid(n_tiles, Hq);
+  dim3 grid(n_tiles, Hq, kv_planes > 2 ? kv_planes - 1 : 1);
   // the largest head size sets the limit once (not per launch: launches may be under stream capture)
   static bool configured = false;
   if (!configured) {
@@ -158,8 +159,8 @@ extern "C" int qe_paged_attention_generic(const void* q, long q_stride, const vo
     if (e != cudaSuccess) QE_REFUSE("paged_attention: shared memory %d: %s", max_smem, cudaGetErrorString(e));
     configured = true;
   }
-  const int planes = kv_planes == 1 ? 1 : 2;
-  if (v_shift < 0 || v_shift >= Hkv || (v_shift && planes == 1)) QE_REFUSE("paged_attention: a shift of %d over %d kv heads", v_shift, Hkv);
+  const int planes = kv_planes;
+  if (planes < 1 || v_shift < 0 || v_shift >= Hkv || (v_shift && planes != 2)) QE_REFUSE("paged_attention: a shift of %d over %d kv heads", v_shift, Hkv);
 #define AGL(TT, DR) qe_launch(attention_generic_kernel<TT, DR>, grid, dim3(AG_WARPS * 32), smem, stream, (const TT*)q, q_stride, \
                               (const TT*)pages, block_tables, max_blocks, cu_q, ctx_lens, tiles, (TT*)out, scale, window, Hq, Hkv, D, \
                               page_size, slopes, planes, softcap, sinks, v_shift)

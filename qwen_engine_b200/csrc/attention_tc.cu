@@ -34,6 +34,9 @@
 // of a held page past the request's length are read as they are and masked, so pages must hold finite
 // values (the cache starts as zeros and only kernels write to it).
 //
+// Values of n blocks of 128 channels (pages of 1 + n planes: keys, then the blocks): a unit is a tile, a kv head and ONE
+// block, so the scores are formed once per block; a head's output has n 128 channels.
+//
 // Every wait on an mbarrier, and the last part's wait for the others' to be written, is bounded: a wait that
 // runs out records a code in a device flag, raises a CTA-wide abort that the other roles see in their own waits, and the CTA skips its stores, frees its
 // tensor memory and returns; the host reads the flag with qe_flash_attention_tc_status().
@@ -56,7 +59,7 @@ static __device__ int g_at_status = 0;          // 0 = fine; else code of the fi
 
 // A work unit (a work item for one kv head) as every role of the CTA sees it.
 struct AtUnit {
-  int req, q0, part, n_parts, split, row0, hkv;
+  int req, q0, part, n_parts, split, row0, hkv, vb;  // hkv: the kv head; vb: the block of values
   int nrows, first_pos, kv_begin, kv_end, kt_first, n_steps;
   bool two;                                         // the second softmax group has rows
 };
@@ -80,6 +83,7 @@ struct AtArgs {
   float cap_in, cap_mul;    // bent scores: the raw score s becomes cap_mul tanh(s cap_in), cap_in = scale / cap, cap_mul = cap / scale (0: as they are)
   const float* sinks;       // null, or float32 [Hq]: exp(sinks[h]) joins head h's denominator (no key, no value)
   int v_shift;              // the weights of a head of kv head c meet the values of kv head (c + v_shift) mod Hkv
+  int vp;                   // blocks of values per kv head (1: values of AT_D channels)
 };
 
 __device__ __forceinline__ uint32_t at_pack(float lo, float hi) {
@@ -137,8 +141,10 @@ __device__ __forceinline__ void at_softmax_sync() { asm volatile("bar.sync 1, %0
 
 __device__ __forceinline__ AtUnit at_unit(const AtArgs& A, int unit) {
   AtUnit U;
-  const int item_idx = unit / A.Hkv;
-  U.hkv = unit - item_idx * A.Hkv;
+  const int item_idx = unit / (A.Hkv * A.vp);
+  U.hkv = unit - item_idx * (A.Hkv * A.vp);
+  U.vb = U.hkv / A.Hkv;
+  U.hkv -= U.vb * A.Hkv;
   const int* it = A.items + (size_t)item_idx * AT_ITEM_INTS;      // (the work lists come from the host's copy, not from a kernel)
   U.req = it[0]; U.q0 = it[1]; U.part = it[4]; U.n_parts = it[5]; U.split = it[6]; U.row0 = it[7];
   const int q_len = it[8], ctx = it[9];
@@ -239,7 +245,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             if (page < 0) page = A.num_pages;       // outside the tensor: the box is filled with zeros
             __nv_bfloat16* dst = (kind ? sm.v[st][half] : sm.k[st][half]) + (size_t)box * box_rows * 64;
             tma_load_5d(dst, &map_kv, kind ? &sm.v_full[st] : &sm.k_full[st], half * 64, y,
-                        kind ? (U.hkv + A.v_shift) % A.Hkv : U.hkv, kind, page);
+                        kind ? (U.hkv + A.v_shift) % A.Hkv : U.hkv, kind ? 1 + U.vb : 0, page);
           }
           if (kind) ++issued_v; else ++issued_k;
           if (kind == 0 && j == 0) {
@@ -425,6 +431,8 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     for (int ui = u_begin; ui < u_end; ++ui) {
       const AtUnit U = unit_at(ui);
       const int n_steps = U.n_steps, hkv = U.hkv, part = U.part;
+      const int HV = Hkv * A.vp, hvb = U.vb * Hkv + hkv;      // (kv head, block of values): what parts and counters are kept by
+      const size_t out_hd = (size_t)AT_D * A.vp;              // a head's channels of the output
       const bool active = w == 0 || U.two;
       const bool valid = r < U.nrows;
       const int pos = valid ? U.first_pos + r / G : -1;
@@ -568,7 +576,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
       // own accumulator never leaving tensor memory; 3: the CTA is giving up.
       int role = 0;
       const bool is_part = part >= 0 && A.counters != nullptr && U.n_parts > 0;
-      int* const arrived = is_part ? A.counters + 2 * ((part - U.split) * Hkv + hkv) : nullptr;     // [1]: parts written
+      int* const arrived = is_part ? A.counters + 2 * ((part - U.split) * HV + hvb) : nullptr;     // [1]: parts written
       if (is_part) {
         if (!ok) sm.abort_flag = 1;
         at_softmax_sync();
@@ -600,7 +608,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
           const float l_all = (A.sinks && valid && part < 0 && l_run > 0.f)
                                   ? l_run + exp2f(A.sinks[hkv * G + r % G] * 1.4426950408889634f - m_run) : l_run;
           const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
-          const size_t slot = part >= 0 ? ((size_t)part * Hkv + hkv) * A.part_rows + r : 0;
+          const size_t slot = part >= 0 ? ((size_t)part * HV + hvb) * A.part_rows + r : 0;
           const int wrow0 = w * AT_ROWS + quarter * 32;       // the warp's first row of the tile
           uint4* stage = sm.stage[warp];
           const int nrows = U.nrows;
@@ -612,9 +620,9 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             if (rr >= nrows) { dst[k] = nullptr; continue; }
             if (part < 0) {
               const int t2 = rr / G, h2 = rr - t2 * G;
-              dst[k] = reinterpret_cast<char*>(A.out + (size_t)(U.row0 + U.q0 + t2) * ((size_t)Hq * AT_D) + (size_t)(hkv * G + h2) * AT_D) + 16 * (lane & 3);
+              dst[k] = reinterpret_cast<char*>(A.out + (size_t)(U.row0 + U.q0 + t2) * (Hq * out_hd) + (hkv * G + h2) * out_hd + U.vb * AT_D) + 16 * (lane & 3);
             } else {
-              dst[k] = reinterpret_cast<char*>(A.part_acc + (((size_t)part * Hkv + hkv) * A.part_rows + rr) * AT_D) + 16 * (lane & 3);
+              dst[k] = reinterpret_cast<char*>(A.part_acc + (((size_t)part * HV + hvb) * A.part_rows + rr) * AT_D) + 16 * (lane & 3);
             }
           }
 #pragma unroll 1
@@ -653,7 +661,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         const int first = part - U.split, me = U.split, n_parts_of_tile = U.n_parts, nrows = U.nrows;
         const int wrow0 = w * AT_ROWS + quarter * 32;
         uint4* stage = sm.stage[warp];
-        const size_t part_stride = (size_t)Hkv * A.part_rows;        // rows between a part and the next
+        const size_t part_stride = (size_t)HV * A.part_rows;        // rows between a part and the next
         auto merged_out = [&](auto p2_tag, auto ch_tag) {
           // P2: the parts, rounded up; CH: columns of the others' accumulators asked for at a time (all loads in flight)
           constexpr int P2 = decltype(p2_tag)::value, CH = decltype(ch_tag)::value, PASSES = CH / 16;
@@ -666,7 +674,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             const int row = 8 * k + (lane >> 2), rr = wrow0 + row;
             const float m_own = __shfl_sync(0xffffffffu, m_run, row), l_own = __shfl_sync(0xffffffffu, l_run, row);
             const bool in = rr < nrows;
-            const size_t sl0 = ((size_t)first * Hkv + hkv) * A.part_rows + rr;
+            const size_t sl0 = ((size_t)first * HV + hvb) * A.part_rows + rr;
             float mm[P2], ll[P2];
 #pragma unroll
             for (int sp = 0; sp < P2; ++sp) {
@@ -690,7 +698,7 @@ flash_attention_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             for (int sp = 0; sp < P2; ++sp) fw[k][sp] *= inv;
             src[k] = in ? A.part_acc + sl0 * AT_D + 4 * (lane & 3) : nullptr;
             const int t2 = rr / G, h2 = rr - t2 * G;
-            outp[k] = in ? reinterpret_cast<char*>(A.out + (size_t)(U.row0 + U.q0 + t2) * ((size_t)Hq * AT_D) + (size_t)(hkv * G + h2) * AT_D) + 8 * (lane & 3)
+            outp[k] = in ? reinterpret_cast<char*>(A.out + (size_t)(U.row0 + U.q0 + t2) * (Hq * out_hd) + (hkv * G + h2) * out_hd + U.vb * AT_D) + 8 * (lane & 3)
                          : nullptr;
           }
           uint32_t o[32];
@@ -876,7 +884,7 @@ extern "C" int qe_flash_attention_tc_supported(int Hq, int Hkv, int D, int page_
 // which the caller has sorted by key steps, longest first, each to the CTA with the least work so far; item_cost[i] is
 // what a unit of item i costs (its key steps plus what its start, its end and, for a part, its scratch and merge
 // cost, in key steps).  out: n_ctas + 1 offsets into out itself, then the CTAs' unit numbers; it must hold
-// n_ctas + 1 + n_items Hkv ints.  Returns the number of ints written, 0 if the arguments make no sense.
+// n_ctas + 1 + n_items Hkv ints.  (With n blocks of values per kv head, Hkv here is the number of (kv head, block) pairs.)  Returns the number of ints written, 0 if the arguments make no sense.
 extern "C" int qe_flash_attention_tc_schedule(const float* item_cost, int n_items, int Hkv, int n_ctas, int* out) {
   if (n_items <= 0 || Hkv <= 0 || n_ctas <= 0) return 0;
   const long n_units = (long)n_items * Hkv;
@@ -925,10 +933,12 @@ extern "C" int qe_flash_attention_tc(const void* q, long q_stride, int T, const 
                                      const int* sched, int n_ctas,
                                      void* out, float* part_acc, float* part_ml, int part_rows, int* counters,
                                      float scale, int window, int Hq, int Hkv, int D, int page_size,
-                                     const float* slopes, float softcap, const float* sinks, int v_shift, cudaStream_t stream) {
+                                     const float* slopes, float softcap, const float* sinks, int v_shift, int value_blocks, cudaStream_t stream) {
   if (n_items <= 0) return 0;
-  if (sched == nullptr || n_ctas <= 0 || (long)n_ctas > (long)n_items * Hkv)
-    QE_REFUSE("flash_attention_tc: a schedule for 1 to %ld CTAs is needed, not one for %d", (long)n_items * Hkv, n_ctas);
+  if (value_blocks < 1 || (value_blocks > 1 && v_shift)) QE_REFUSE("flash_attention_tc: %d blocks of values, a shift of %d", value_blocks, v_shift);
+  const long n_units = (long)n_items * Hkv * value_blocks;
+  if (sched == nullptr || n_ctas <= 0 || (long)n_ctas > n_units)
+    QE_REFUSE("flash_attention_tc: a schedule for 1 to %ld CTAs is needed, not one for %d", n_units, n_ctas);
   if (part_acc && part_rows != 2 * AT_ROWS) QE_REFUSE("flash_attention_tc: parts have %d rows, not %d", part_rows, 2 * AT_ROWS);
   if (!qe_flash_attention_tc_supported(Hq, Hkv, D, page_size))
     QE_REFUSE("flash_attention_tc: heads %d/%d, head_dim %d, page size %d are not supported", Hq, Hkv, D, page_size);
@@ -937,7 +947,7 @@ extern "C" int qe_flash_attention_tc(const void* q, long q_stride, int T, const 
   if (scale <= 0.f) QE_REFUSE("flash_attention_tc: the scale must be positive");
   if (v_shift < 0 || v_shift >= Hkv) QE_REFUSE("flash_attention_tc: a shift of %d over %d kv heads", v_shift, Hkv);
   if (slopes && softcap > 0.f) QE_REFUSE("flash_attention_tc: scores are biased by distance or bent, not both");
-  if ((long)n_items * Hkv > 0x7fffffffL) QE_REFUSE("flash_attention_tc: too many work items");
+  if (n_units > 0x7fffffffL) QE_REFUSE("flash_attention_tc: too many work items");
   const int G = Hq / Hkv;
   CUtensorMap map_q, map_kv;
   {
@@ -948,8 +958,9 @@ extern "C" int qe_flash_attention_tc(const void* q, long q_stride, int T, const 
   }
   {
     const uint64_t P = (uint64_t)page_size;
-    const uint64_t dims[5] = {(uint64_t)AT_D, P, (uint64_t)Hkv, 2, (uint64_t)num_pages};
-    const uint64_t strides[4] = {(uint64_t)AT_D * 2, P * AT_D * 2, (uint64_t)Hkv * P * AT_D * 2, 2ull * Hkv * P * AT_D * 2};
+    const uint64_t planes = 1 + (uint64_t)value_blocks;
+    const uint64_t dims[5] = {(uint64_t)AT_D, P, (uint64_t)Hkv, planes, (uint64_t)num_pages};
+    const uint64_t strides[4] = {(uint64_t)AT_D * 2, P * AT_D * 2, (uint64_t)Hkv * P * AT_D * 2, planes * Hkv * P * AT_D * 2};
     const uint32_t box[5] = {64, (uint32_t)(page_size < AT_BN ? page_size : AT_BN), 1, 1, 1};
     if (!qe_tensor_map_bf16(pages, 5, dims, strides, box, &map_kv)) return 1;
   }
@@ -957,7 +968,7 @@ extern "C" int qe_flash_attention_tc(const void* q, long q_stride, int T, const 
   while ((1 << page_shift) < page_size) ++page_shift;
   AtArgs args{block_tables, max_blocks, num_pages, items, sched, (__nv_bfloat16*)out, part_acc, part_ml, part_rows, counters,
               scale * 1.4426950408889634f, window, Hq, Hkv, page_shift, slopes, 1.f / scale,
-              softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f, sinks, v_shift};
+              softcap > 0.f ? scale / softcap : 0.f, softcap > 0.f ? softcap / scale : 0.f, sinks, v_shift, value_blocks};
   const size_t smem = sizeof(AtSmem) + 1024;
   static bool configured = false;
   if (!configured) {

@@ -147,6 +147,8 @@ class DecoderModel:
         self.embed = ops.prepare_matrix(source.get(lo.embed_name).to(dtype).to(device))
         for ls, block in zip(lo.layers, self.blocks):
             block.load(ls.weight_prefix, source, dtype, device)
+            if block.mixer.output_bias() is not None and not block.adds_output_bias:
+                raise ValueError(f"{ls.weight_prefix}: block {ls.block.name!r} does not add the bias of its mixer's result")
         self.final_norm.load(lo.final_norm_prefix, source, dtype, device)
         if self.embed_norm is not None:
             self.embed_norm.load(lo.embed_norm_prefix, source, dtype, device)
@@ -232,12 +234,15 @@ class DecoderModel:
             ctx.extras["norm_after_block"] = self.blocks[nxt].first_norm() if nxt is not None else None
             if history is not None:
                 history.run = i
+            if not self.blocks[entry.layer].takes_second:
+                stream.fold_second()
             self.blocks[entry.layer].forward(ctx, stream, view, group, entry.write_cache)
             if not self.blocks[entry.layer].keeps_copy:
                 stream.copy_current = False
         ctx.extras["next_cache"] = ctx.extras["weights_after_ffn"] = ctx.extras["norm_after_block"] = None
         if ctx.num_logit_rows == 0:
             return None
+        stream.fold_second()
         N = ctx.num_logit_rows
         normed = ctx.arena.alloc((N, H), ctx.dtype)
         self.final_norm.add_norm_rows(ctx, stream.resid, stream.delta if stream.has_delta else None,

@@ -260,6 +260,8 @@ class ResidualStream:
     ``has_delta`` set, to be added by the next norm.  ``ssq`` [T, P] float32 holds ``n_ssq`` partial
     sums of squares of every row of ``resid`` when the kernel that last wrote the stream left them
     (``n_ssq`` = 0: unknown); a norm fused into the next product starts from them.
+    ``second`` [T, H]: for arrangements whose two sublayers run side by side, the other branch's output (``has_second``),
+    where neither could be added at once (``second_buffer`` makes room, ``fold_second`` adds it for a reader that takes one).
     ``copy`` [T, H]: for arrangements whose sublayers read the stream itself, its rows rounded to the compute type
     (None in float32, where the stream serves as it is), up to date while ``copy_current``: the kernels that write the
     stream for such an arrangement leave it behind."""
@@ -270,6 +272,19 @@ class ResidualStream:
         self.has_delta = False
         self.n_ssq = 0
         self.copy_current = False
+        self.second: Optional[torch.Tensor] = None
+        self.has_second = False
+
+    def second_buffer(self, alloc_step) -> torch.Tensor:
+        """Room for a second pending branch output, for the rest of the step."""
+        if self.second is None:
+            self.second = alloc_step(tuple(self.delta.shape), self.delta.dtype)
+        return self.second
+
+    def fold_second(self) -> None:
+        if self.has_second:
+            scaled_add(self.resid, self.second, 1.0)
+            self.has_second, self.n_ssq = False, 0
 
     def rounded(self) -> torch.Tensor:
         """The stream's rows in the compute type (the stream itself in float32)."""
@@ -976,9 +991,27 @@ def split_geometry(geo) -> tuple:
 
 
 def geometry_planes(geo) -> int:
-    """The sixth entry of a geometry, if it has one: 1 for a cache whose pages hold one plane per kv head, the values
-    being the keys' channels (a latent cache; the tcgen05 kernel does not take it), else 2."""
+    """The sixth entry of a geometry, if it has one: the planes of a cache page.  1: the values are the keys' channels (a
+    latent cache; a tcgen05 kernel of its own); 2: keys and values; 1 + n: keys and n blocks of ``head size`` value
+    channels (values of n times the keys' size)."""
     return int(geo[5]) if len(geo) > 5 else 2
+
+
+def value_blocks(geo) -> int:
+    """How many blocks of ``head size`` value channels a kv head has (the attention kernels run once per block)."""
+    return max(1, geometry_planes(geo) - 1)
+
+
+def value_block_size(key_dim: int, value_dim: int) -> tuple[int, int]:
+    """(D, n): the head size the cache and the attention kernels see, and how many blocks of D value channels a head has,
+    for keys of ``key_dim`` and values of ``value_dim`` channels.  Keys are padded up to D, values up to n D.  Values that are
+    larger than keys which fit 128 channels come in blocks of 128 (the head size of the fastest kernels); otherwise one
+    block serves, of the larger of the two sizes."""
+    def up(x):
+        return -(-x // 16) * 16
+    if key_dim <= 128 < value_dim:
+        return 128, -(-value_dim // 128)
+    return up(max(key_dim, value_dim)), 1
 
 
 def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
@@ -1008,10 +1041,11 @@ def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
         G = Hq // Hkv
         tpt = FLASH_ROWS // G
         latent_tc = latent_tc_supported(geo, dtype, page_size)
-        use_tc = uniform_splits is None and (latent_tc or (geometry_planes(geo) == 2 and tc_attention_supported(dtype, Hq, Hkv, D, page_size)))
+        vb = value_blocks(geo)
+        use_tc = uniform_splits is None and (latent_tc or (geometry_planes(geo) >= 2 and tc_attention_supported(dtype, Hq, Hkv, D, page_size)))
         on_tc = [use_tc and n * G >= TC_MIN_ROWS for n in q_lens]
         tc_tiles: list = []
-        base = sum(-(-n // tpt) for n, tc in zip(q_lens, on_tc) if not tc) * Hkv
+        base = sum(-(-n // tpt) for n, tc in zip(q_lens, on_tc) if not tc) * Hkv * vb
         items: list[int] = []
         merge: list[int] = []
         n_parts, part_rows, row0, max_rows = 0, 1, 0, 0
@@ -1058,7 +1092,7 @@ def plan_attention(q_lens: list[int], ctx_lens: list[int], page_size: int,
             plan[f"tc{gi}_items"] = [x for _, lo, hi, (r, q0, first, n, c) in tc_tiles for x in (r, q0, lo, hi, -1, 0, 0, first, n, c, 0, 0)]
             plan[f"tc{gi}_info"] = [0, LATENT_TC_ROWS, len(tc_tiles)]
         elif tc_tiles:
-            tc_items, tc_parts, tc_sched, tc_ctas = _plan_tc_tiles(tc_tiles, Hkv)
+            tc_items, tc_parts, tc_sched, tc_ctas = _plan_tc_tiles(tc_tiles, Hkv * vb)
             plan[f"tc{gi}_items"] = tc_items
             plan[f"tc{gi}_sched"] = tc_sched
             plan[f"tc{gi}_info"] = [tc_parts, TC_ROWS, tc_ctas]
@@ -1076,6 +1110,8 @@ def decode_splits(num_reqs: int, max_tokens: int, geometries, dtype: torch.dtype
         Hq, Hkv, D, window, _ = split_geometry(geo)
         span = min(max_tokens, window) if window else max_tokens
         target = FLASH_TARGET_CTAS
+        Hkv *= value_blocks(geo)                            # (one CTA per kv head and block of values)
+        Hq *= value_blocks(geo)
         if latent_decode_supported(geo, dtype):
             # one CTA per SM; the parts of a request form a cluster (as many of 8, 4, 2 as fit on chip, keep every CTA on the
             # GPU at once and leave each part enough keys)
@@ -1172,6 +1208,7 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
     one plane bent scores and sinks only).
     ``value_shifts`` S > 1: out is [S, T, Hq D] and entry s is the output for shift s; where the whole step is served by
     the kernels for few rows, the shifts are one launch (a grid dimension), else one launch each.
+    Pages of 1 + n planes, n > 1: a kv head has n blocks of D value channels, and out is [T, Hq n D].
     ``value_dim`` (a cache of one plane): only so many of a key's first channels are its value; what the output holds
     behind them is not defined.
 
@@ -1180,7 +1217,11 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
     Hq, Hkv, D = num_heads, num_kv_heads, head_dim
     T = qkv.shape[0]
     S = int(value_shifts)
-    if S > 1:
+    VB = max(1, int(kv_pages.shape[1]) - 1) if kv_pages.dim() == 5 else 1     # blocks of values per kv head
+    if VB > 1:
+        _need(S == 1 and value_shift == 0 and slopes is None, "paged_attention: several blocks of values go without shifts and a distance bias")
+        _need(out.shape == (T, Hq * VB * D) and out.is_contiguous() and out.dtype == qkv.dtype, "paged_attention: out must be [T, Hq n D] for n blocks of values")
+    elif S > 1:
         _need(value_shift == 0 and S <= Hkv and out.shape == (S, T, Hq * D) and out.is_contiguous() and out.dtype == qkv.dtype,
               "paged_attention: several shifts write out [S, T, Hq D], S <= Hkv")
         plan0 = ctx.attn_plan
@@ -1193,8 +1234,8 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
             return
     else:
         _need(out.shape == (T, Hq * D) and out.is_contiguous() and out.dtype == qkv.dtype, "paged_attention: out must be [T, Hq D]")
-    _need(kv_pages.dtype == qkv.dtype and kv_pages.dim() == 5 and kv_pages.is_contiguous() and kv_pages.shape[1] in (1, 2),
-          "paged_attention: kv_pages must be [pages, 2 (or 1: the values are the keys' channels), Hkv, page, D] in q's dtype")
+    _need(kv_pages.dtype == qkv.dtype and kv_pages.dim() == 5 and kv_pages.is_contiguous() and kv_pages.shape[1] >= 1,
+          "paged_attention: kv_pages must be [pages, 2 (1: the values are the keys' channels; 1 + n: n blocks of values), Hkv, page, D] in q's dtype")
     planes = int(kv_pages.shape[1])
     _i32(block_tables, "block_tables")
     global last_attention_kernel
@@ -1207,10 +1248,12 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
         _need(sinks.dtype == torch.float32 and sinks.numel() == Hq and sinks.is_contiguous(), "paged_attention: sinks must be float32 [Hq]")
     if plain:
         _need(slopes is None and 0 <= value_shift < Hkv, "paged_attention: bent scores, sinks and shifted values go without a distance bias")
-        _need(planes == 2 or (value_shift == 0 and S == 1), "paged_attention: shifted values go with a cache of two planes")
+        _need(planes >= 2 or (value_shift == 0 and S == 1), "paged_attention: shifted values go with a cache of two planes")
     if planes == 1:
         _need(slopes is None, "paged_attention: no distance bias over a cache of one plane")
         key = index.get((Hq, Hkv, D, window, False, 1))
+    elif planes > 2:
+        key = index.get((Hq, Hkv, D, window, False, planes))
     else:
         key = index.get((Hq, Hkv, D, window, True)) if slopes is not None else index.get((Hq, Hkv, D, window), index.get((Hq, Hkv, D, window, False)))
     _need(value_dim is None or (planes == 1 and 1 <= value_dim <= D), "paged_attention: a value size of its own goes with a cache of one plane")
@@ -1228,16 +1271,16 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
         tc_parts, tc_rows, tc_ctas = plan[f"tc{key}_info_host"]
         part_acc = part_ml = counters = None
         if tc_parts:
-            _need(2 * tc_parts * Hkv <= _MERGE_COUNTERS, "paged_attention: too many parts")   # (two counters a tile and kv head)
-            part_acc = ctx.arena.alloc((tc_parts * Hkv * tc_rows, D), torch.float32)
-            part_ml = ctx.arena.alloc((tc_parts * Hkv * tc_rows, 2), torch.float32)
+            _need(2 * tc_parts * Hkv * VB <= _MERGE_COUNTERS, "paged_attention: too many parts")   # (two counters a tile and kv head)
+            part_acc = ctx.arena.alloc((tc_parts * Hkv * VB * tc_rows, D), torch.float32)
+            part_ml = ctx.arena.alloc((tc_parts * Hkv * VB * tc_rows, 2), torch.float32)
             counters = _merge_counters(qkv.device, "tc")
         _check(lib().qe_flash_attention_tc(
             _ptr(qkv), ctypes.c_long(qkv.stride(0)), T, _ptr(kv_pages), int(kv_pages.shape[0]), _ptr(block_tables),
             int(block_tables.shape[1]), _ptr(tc_items), tc_items.numel() // FLASH_ITEM_INTS,
             _ptr(plan[f"tc{key}_sched"]), int(tc_ctas), _ptr(out),
             _ptr(part_acc), _ptr(part_ml), int(tc_rows), _ptr(counters), ctypes.c_float(scale), int(window),
-            Hq, Hkv, D, int(kv_pages.shape[3]), _ptr(slopes), ctypes.c_float(softcap), _ptr(sinks), int(value_shift), _stream()),
+            Hq, Hkv, D, int(kv_pages.shape[3]), _ptr(slopes), ctypes.c_float(softcap), _ptr(sinks), int(value_shift), VB, _stream()),
             "flash_attention_tc")
     if key is not None and f"fa{key}_items" in plan:
         items, merge = plan[f"fa{key}_items"], plan[f"fa{key}_merge"]
@@ -1246,6 +1289,10 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
         if n_items == 0 and f"tc{key}_items" in plan:
             return                      # every request of the step went to the kernel above
         part_acc = part_ml = None
+        shift_out = T * Hq * D
+        if VB > 1:                      # the blocks of values run where shifts of the values' kv head would (a grid dimension)
+            S, shift_out = VB, D
+            _need(S * n_parts * Hkv <= _MERGE_COUNTERS, "paged_attention: too many parts")
         if n_parts:
             part_acc = ctx.arena.alloc((S * n_parts * Hkv * part_rows, D), torch.float32)
             part_ml = ctx.arena.alloc((S * n_parts * Hkv * part_rows, 2), torch.float32)
@@ -1281,7 +1328,7 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
                 _ptr(items), n_items, _ptr(out), _ptr(part_acc), _ptr(part_ml), int(part_rows), _ptr(counters),
                 int(max_rows), cluster, int(DECODE_ATTENTION_MMA_WIDE and n_items * Hkv * S <= TC_TARGET_CTAS),
                 ctypes.c_float(scale), int(window), Hq, Hkv, D, int(kv_pages.shape[3]), _ptr(slopes), planes,
-                ctypes.c_float(softcap), _ptr(sinks), int(value_shift), S, ctypes.c_long(T * Hq * D), int(n_parts), _stream()),
+                ctypes.c_float(softcap), _ptr(sinks), int(value_shift), S, ctypes.c_long(shift_out), int(n_parts), _stream()),
                 "decode_attention_mma")
             return
         last_attention_kernel = "flash_attention"
@@ -1290,7 +1337,7 @@ def paged_attention(qkv: torch.Tensor, kv_pages: torch.Tensor, block_tables: tor
             _ptr(ctx.cu_q), _ptr(ctx.ctx_lens), _ptr(items), n_items, _ptr(merge), n_merge, _ptr(out),
             _ptr(part_acc), _ptr(part_ml), int(part_rows), _ptr(counters), int(small_tiles), ctypes.c_float(scale), int(window),
             Hq, Hkv, D, int(kv_pages.shape[3]), _ptr(slopes), planes, ctypes.c_float(softcap), _ptr(sinks), int(value_shift),
-            S, ctypes.c_long(T * Hq * D), int(n_parts), _stream()), "flash_attention")
+            S, ctypes.c_long(shift_out), int(n_parts), _stream()), "flash_attention")
         return
     tiles = plan["tiles"]
     n_tiles = tiles.numel() // 2
@@ -1860,6 +1907,165 @@ def head_mix_gate(partial: torch.Tensor, mix: Optional[torch.Tensor], gate: Opti
     _check(lib().qe_head_mix_gate(_ptr(partial), ctypes.c_long(T * H * D), S, _ptr(mix), _ptr(gate),
                                   ctypes.c_long(gate.stride(0) if gate is not None else 0), _ptr(out), ctypes.c_long(out.stride(0)),
                                   T, H, Hkv, D, _dt(out), _stream()), "head_mix_gate")
+
+
+def add_rmsnorm_pair(resid: torch.Tensor, delta_a: Optional[torch.Tensor], delta_b: Optional[torch.Tensor], bias: Optional[torch.Tensor],
+                     w1: torch.Tensor, out1: torch.Tensor, w2: Optional[torch.Tensor], out2: Optional[torch.Tensor], eps: float) -> None:
+    """What two sublayers side by side read of the float32 stream: x = resid + delta_a + delta_b (each may be None); out1 =
+    rmsnorm(x) * w1 and, where given, out2 = rmsnorm(x) * w2, the root mean square formed once; resid = x + bias (a bias
+    that the sublayers' results carry; it joins the stream here, behind the norms).  resid, w1, w2, bias float32."""
+    T, H = resid.shape
+    _need(resid.dtype == torch.float32 and resid.is_contiguous(), "add_rmsnorm_pair: resid must be contiguous float32")
+    for w in (w1, w2, bias):
+        _need(w is None or (w.dtype == torch.float32 and w.shape == (H,) and w.is_contiguous()), "add_rmsnorm_pair: weights and bias must be float32 [H]")
+    for t in (out1, out2, delta_a, delta_b):
+        _need(t is None or (t.shape == (T, H) and t.is_contiguous() and t.dtype == out1.dtype), "add_rmsnorm_pair: outputs and deltas must be contiguous [T, H] of one type")
+    _need((w2 is None) == (out2 is None), "add_rmsnorm_pair: a second output comes with its weights")
+    _check(lib().qe_add_rmsnorm_pair(_ptr(resid), _ptr(delta_a), _ptr(delta_b), _ptr(bias), _ptr(w1), _ptr(w2), ctypes.c_float(eps),
+                                     _ptr(out1), _ptr(out2), T, H, _dt(out1), _stream()), "add_rmsnorm_pair")
+
+
+def group_norm_gate(x: torch.Tensor, gate: Optional[torch.Tensor], weight: torch.Tensor, eps: float, groups: int, out: torch.Tensor,
+                    gate_kind: Optional[str] = "silu", gate_first: bool = False, divisor: Optional[torch.Tensor] = None,
+                    scale: float = 1.0) -> None:
+    """A recurrent mixer's output normed in ``groups`` equal parts and gated: out = y / rms(y) * weight * g(gate) * scale per
+    part, with y = x / divisor (float32 [T, groups], optional).  ``gate_first``: the gate comes ahead of the norm, y = x *
+    g(gate).  x float32 [T, C], weight float32 [C], gate and out [T, C] in the compute type; rows of x, gate and out may
+    be strided."""
+    T, C = x.shape
+    G = int(groups)
+    _need(gate_kind in _GATES, f"group_norm_gate: unknown gate {gate_kind!r}")
+    for t, name in ((x, "x"), (out, "out")) + (((gate, "gate"),) if gate is not None else ()):
+        _rows(t, f"group_norm_gate: {name}")
+        _need(t.shape == (T, C), f"group_norm_gate: {name} must be [T, C]")
+    _need(G >= 1 and C % G == 0, f"group_norm_gate: {C} channels do not split into {G} equal parts")
+    _need(x.dtype == torch.float32 and (gate is None or gate.dtype == out.dtype), "group_norm_gate: x must be float32, gate in out's dtype")
+    _need(weight.dtype == torch.float32 and weight.shape == (C,) and weight.is_contiguous(), "group_norm_gate: weight must be float32 [C]")
+    _need(divisor is None or (divisor.dtype == torch.float32 and divisor.shape == (T, G) and divisor.is_contiguous()),
+          "group_norm_gate: the divisors must be float32 [T, groups]")
+    _check(lib().qe_group_norm_gate(_ptr(x), ctypes.c_long(x.stride(0)), _ptr(gate), ctypes.c_long(gate.stride(0) if gate is not None else 0),
+                                    _ptr(weight), _ptr(divisor), ctypes.c_float(eps), _ptr(out), ctypes.c_long(out.stride(0)),
+                                    ctypes.c_float(scale), _GATES[gate_kind if gate is not None else None], int(bool(gate_first)),
+                                    T, G, C // G, _dt(out), _stream()), "group_norm_gate")
+
+
+def _conv_operands(name: str, x: torch.Tensor, in_bias, w, state, C: int) -> int:
+    """The checks the two convolutions share; returns the number of taps."""
+    _rows(x, f"{name}: x")
+    _need(x.shape[1] == C, f"{name}: x must have {C} columns")
+    taps = 1 if w is None else int(w.shape[0])
+    _need(w is None or (w.dtype == torch.float32 and w.shape == (taps, C) and w.is_contiguous()), f"{name}: w must be float32 [taps, C]")
+    _need(in_bias is None or (in_bias.dtype == torch.float32 and in_bias.shape == (C,) and in_bias.is_contiguous()), f"{name}: the bias must be float32 [C]")
+    if taps > 1:
+        _need(state is not None and state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (taps - 1, C),
+              f"{name}: state must be float32 [slots, taps - 1, C]")
+    return taps
+
+
+def conv_act(x: torch.Tensor, w: Optional[torch.Tensor], state: Optional[torch.Tensor], ctx, out: torch.Tensor,
+             in_bias: Optional[torch.Tensor] = None, out_bias: Optional[torch.Tensor] = None, silu: bool = True,
+             write_state: bool = True) -> None:
+    """A short causal convolution over the tokens of each request, channel by channel: with u = x + in_bias,
+    out[t, c] = act(sum_j w[j, c] u[t - (taps - 1) + j, c] + out_bias[c]), act silu or none, rounded once.  x [T, C] and
+    out [T, C] in the compute type (rows may be strided); w float32 [taps, C] (None: one tap of weight 1); state float32
+    [slots, taps - 1, C] holds each request's last taps - 1 rows u (zeros count before its first token) and is moved on."""
+    C = x.shape[1]
+    taps = _conv_operands("conv_act", x, in_bias, w, state, C)
+    _rows(out, "conv_act: out")
+    _need(out.shape == x.shape and out.dtype == x.dtype, "conv_act: out must be [T, C] in x's dtype")
+    _need(out_bias is None or (out_bias.dtype == torch.float32 and out_bias.shape == (C,) and out_bias.is_contiguous()), "conv_act: out_bias must be float32 [C]")
+    _check(lib().qe_conv_act(_ptr(x), ctypes.c_long(x.stride(0)), _ptr(in_bias), _ptr(w), _ptr(state if taps > 1 else None), _ptr(ctx.cu_q),
+                             _ptr(ctx.ctx_lens), _ptr(ctx.slot_ids), _ptr(out_bias), _ptr(out), ctypes.c_long(out.stride(0)), int(ctx.num_reqs),
+                             int(ctx.max_q_len), C, taps, int(bool(write_state)), int(bool(silu)), _dt(x), _stream()), "conv_act")
+
+
+def conv_qkv(x: torch.Tensor, w: Optional[torch.Tensor], state: Optional[torch.Tensor], ctx, q: torch.Tensor, kv_pages: torch.Tensor,
+             slot_mapping: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, in_bias: Optional[torch.Tensor] = None,
+             inv_freq: Optional[torch.Tensor] = None, rotary_dim: int = 0, cos_sin: Optional[torch.Tensor] = None,
+             write_kv: bool = True) -> None:
+    """What attention does per token between its projection and the attention kernel, where q, k and v pass a short causal
+    convolution on each channel: x [T, (Hq + Hkv + Hkv n) D] (rows may be strided) holds the query heads, the key heads and
+    every kv head's n blocks of D value channels.  u = x + in_bias; y = sum_j w[j] u[t - (taps - 1) + j] (w float32 [taps,
+    columns]; None: y = u); the first ``rotary_dim`` channels of query and key heads turn (half-split pairs, angle position x
+    inv_freq; ``cos_sin`` float32 [T, rotary_dim / 2, 2] if the step has a table of them); q goes to ``q`` [T, Hq D], k and v
+    to the slots of ``slot_mapping`` in ``kv_pages`` [pages, 1 + n, Hkv, page, D].  state float32 [slots, taps - 1, columns]
+    as for ``conv_act``; without ``write_kv`` neither pages nor state change."""
+    T = x.shape[0]
+    Hq, Hkv, D = num_heads, num_kv_heads, head_dim
+    _need(kv_pages.dim() == 5 and kv_pages.shape[1] >= 2 and kv_pages.shape[2] == Hkv and kv_pages.shape[4] == D and kv_pages.is_contiguous()
+          and kv_pages.dtype == x.dtype, "conv_qkv: kv_pages must be [pages, 1 + n, Hkv, page, D] in x's dtype")
+    n = int(kv_pages.shape[1]) - 1
+    taps = _conv_operands("conv_qkv", x, in_bias, w, state, (Hq + Hkv * (1 + n)) * D)
+    _rows(q, "conv_qkv: q")
+    _need(q.shape == (T, Hq * D) and q.dtype == x.dtype, "conv_qkv: q must be [T, Hq D] in x's dtype")
+    _i32(ctx.positions, "positions")
+    if write_kv:
+        _i32(slot_mapping, "slot_mapping")
+        _need(slot_mapping.numel() >= T, "conv_qkv: one cache slot per token")
+    if inv_freq is None:
+        rotary_dim, cos_sin = 0, None
+    else:
+        _need(inv_freq.dtype == torch.float32 and inv_freq.numel() == rotary_dim // 2, "conv_qkv: inv_freq must be float32 [rotary_dim / 2]")
+        _need(cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.shape == (T, rotary_dim // 2, 2) and cos_sin.is_contiguous()),
+              "conv_qkv: cos_sin must be float32 [T, rotary_dim / 2, 2]")
+    _check(lib().qe_conv_qkv(_ptr(x), ctypes.c_long(x.stride(0)), _ptr(in_bias), _ptr(w), _ptr(state if taps > 1 else None), _ptr(ctx.cu_q),
+                             _ptr(ctx.ctx_lens), _ptr(ctx.slot_ids), _ptr(ctx.positions), _ptr(inv_freq), _ptr(cos_sin), int(rotary_dim),
+                             _ptr(q), ctypes.c_long(q.stride(0)), _ptr(kv_pages if write_kv else None), _ptr(slot_mapping if write_kv else None),
+                             int(ctx.num_reqs), int(ctx.max_q_len), Hq, Hkv, n, D, int(kv_pages.shape[3]), taps, int(bool(write_kv)), _dt(x),
+                             _stream()), "conv_qkv")
+
+
+def _memory_scan(q, k, v, state, mstate, ctx, out, den, gates, biases, log_rate, skip, cap, q_scale, den_eps, form, H, G, dk, dv, write_state):
+    T = q.shape[0]
+    for t, name, width in ((q, "q", G * dk), (k, "k", G * dk), (v, "v", H * dv)):
+        _rows(t, f"memory_scan: {name}")
+        _need(t.shape == (T, width) and t.dtype == q.dtype, f"memory_scan: {name} must be [T, {width}] in one type")
+    rows = dv + (1 if form == 1 else 0)
+    _need(state.dtype == torch.float32 and state.is_contiguous() and tuple(state.shape[1:]) == (H, rows, dk),
+          "memory_scan: state must be float32 [slots, H, value channels, dk]")
+    _need(out.shape == (T, H * dv) and out.dtype == torch.float32 and out.is_contiguous(), "memory_scan: out must be float32 [T, H dv]")
+    g0, g1 = gates[0], gates[1] if len(gates) > 1 else None
+    for g in gates:
+        _rows(g, "memory_scan: gates")
+        _need(g.shape == (T, H) and g.dtype in (q.dtype, torch.float32) and g.dtype == g0.dtype, "memory_scan: gates must be [T, H], float32 or the compute type")
+    for t in (*biases, log_rate, skip):
+        _need(t is None or (t.dtype == torch.float32 and t.shape == (H,) and t.is_contiguous()), "memory_scan: per-head constants must be float32 [H]")
+    b0, b1 = biases[0], biases[1] if len(biases) > 1 else None
+    _check(lib().qe_memory_scan(
+        _ptr(q), ctypes.c_long(q.stride(0)), _ptr(k), ctypes.c_long(k.stride(0)), _ptr(v), ctypes.c_long(v.stride(0)), _ptr(state), _ptr(mstate),
+        _ptr(ctx.cu_q), _ptr(ctx.ctx_lens), _ptr(ctx.slot_ids), _ptr(out), _ptr(den), _ptr(g0), ctypes.c_long(g0.stride(0)), _ptr(g1),
+        ctypes.c_long(g1.stride(0) if g1 is not None else 0), int(g0.dtype == torch.float32), _ptr(b0), _ptr(b1), _ptr(log_rate), _ptr(skip),
+        ctypes.c_float(cap), ctypes.c_float(q_scale), ctypes.c_float(den_eps), form, int(ctx.num_reqs), int(ctx.max_q_len), H, G, dk, dv,
+        int(bool(write_state)), _dt(q), _stream()), "memory_scan")
+
+
+def state_space_scan(x: torch.Tensor, B: torch.Tensor, C: torch.Tensor, dt: torch.Tensor, dt_bias: Optional[torch.Tensor], log_rate: torch.Tensor,
+                     skip: Optional[torch.Tensor], state: torch.Tensor, ctx, out: torch.Tensor, num_heads: int, num_groups: int,
+                     state_dim: int, value_dim: int, write_state: bool = True) -> None:
+    """The recurrence of a state-space model with one decay per head and token, over the step's tokens of every request:
+    d = softplus(dt + dt_bias); S <- exp(-exp(log_rate_h) d) S + d B x^T; out = S^T C + skip_h x, per head, S: N x P.
+    x [T, H P], B and C [T, G N] (head h reads group h // (H / G)) and dt [T, H] in the compute type (rows may be strided);
+    state float32 [slots, H, P, N]; out float32 [T, H P]."""
+    _memory_scan(C, B, x, state, None, ctx, out, None, (dt,), (dt_bias,), log_rate, skip, 0.0, 1.0, 0.0, 0, num_heads, num_groups,
+                 state_dim, value_dim, write_state)
+
+
+def matrix_memory_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate_in: torch.Tensor, gate_keep: torch.Tensor,
+                       bias_in: Optional[torch.Tensor], bias_keep: Optional[torch.Tensor], cap: float, state: torch.Tensor,
+                       maxima: torch.Tensor, ctx, out: torch.Tensor, divisor: torch.Tensor, q_scale: float, den_eps: float,
+                       num_heads: int, key_dim: int, value_dim: int, write_state: bool = True) -> None:
+    """A matrix memory with exponential gates, over the step's tokens of every request: i = cap tanh((gate_in + bias_in) / cap),
+    f = logsigmoid(cap tanh((gate_keep + bias_keep) / cap)), m_t = max(f + m_(t-1), i) from m = 0; S <- exp(f + m_(t-1) - m_t) S
+    + exp(i - m_t) k v^T and n alike with k alone; out = S^T q q_scale, and divisor[t, h] = max(|n . q q_scale|, exp(-m_t)) +
+    den_eps, which the head's output is still to be divided by.  q, k [T, H dk], v [T, H dv], gates [T, H] in the compute
+    type (rows may be strided; the gates may be float32); state float32 [slots, H, dv + 1, dk] (the last row is n), maxima
+    float32 [slots, H, dv + 1]; out float32 [T, H dv], divisor float32 [T, H]."""
+    _need(maxima.dtype == torch.float32 and maxima.is_contiguous() and tuple(maxima.shape[1:]) == (num_heads, value_dim + 1),
+          "matrix_memory_scan: maxima must be float32 [slots, H, dv + 1]")
+    _need(divisor.shape == (q.shape[0], num_heads) and divisor.dtype == torch.float32 and divisor.is_contiguous(),
+          "matrix_memory_scan: divisor must be float32 [T, H]")
+    _memory_scan(q, k, v, state, maxima, ctx, out, divisor, (gate_in, gate_keep), (bias_in, bias_keep), None, None, cap, q_scale, den_eps, 1,
+                 num_heads, num_heads, key_dim, value_dim, write_state)
 
 
 def argmax(logits: torch.Tensor, out: torch.Tensor) -> None:

@@ -38,6 +38,13 @@ Options that other designs use (all off for Qwen3):
   the blended v is what is cached.  The kept values are as projected (the keeping layer blends nothing).
 * a position encoding with ``row_permutation()`` (pairs that the kernels do not rotate as stored): the rows of W_q
   and W_k are reordered within every head at load; ``magnitude`` multiplies its cosines and sines.
+* ``conv_taps`` = n: q, k and v each pass a short causal convolution over n tokens on each channel, behind the projection
+  (and its bias) and ahead of the rotation; the last n - 1 projected rows are state of the request (a second cache).
+  ``projection_bias``: biases of the q, k and v projections.  With either, one kernel (``ops.conv_qkv``) takes the
+  projected rows to rotated queries and to the cache; values larger than keys come in blocks of the keys' size
+  (``ops.value_block_size``), so that the cache pads neither; and a window, bent scores, sinks and a sigmoid gate per channel
+  go together.
+* ``output_bias``: a bias of the output projection, which the arrangement adds (``Mixer.output_bias``).
 * ``names``: the tensors' names in the checkpoint.
 """
 from __future__ import annotations
@@ -47,13 +54,14 @@ from typing import Optional
 import torch
 
 from .. import ops
-from ..cache.spec import PagedKVSpec
+from ..cache.spec import FixedStateSpec, PagedKVSpec
 from ..weights.spec import MATRIX, NORM, VECTOR, WeightSpec
 from .base import Mixer, PartSpec, StepContext, register, step_hint
 
 _NAMES = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", out="o_proj.weight",
               q_norm="q_norm.weight", k_norm="k_norm.weight", gate="g_proj.weight",
-              q_bias="q_proj.bias", k_bias="k_proj.bias", sink="sinks", head_mix="head_mix", value_mix="value_mix")
+              q_bias="q_proj.bias", k_bias="k_proj.bias", v_bias="v_proj.bias", out_bias="o_proj.bias", q_conv="q_conv.weight",
+              k_conv="k_conv.weight", v_conv="v_conv.weight", sink="sinks", head_mix="head_mix", value_mix="value_mix")
 
 
 def _pad_rows(w: torch.Tensor, heads: int, dim: int, padded: int) -> torch.Tensor:
@@ -75,7 +83,8 @@ class GQAAttention(Mixer):
                  value_dim: Optional[int] = None, distance_slopes=None, output_gate: Optional[str] = None,
                  names: Optional[dict] = None, tied_values: bool = False, qk_bias: bool = False,
                  query_temperature=None, softcap: Optional[float] = None, sink: bool = False, head_mixing: bool = False,
-                 value_mix: Optional[str] = None):
+                 value_mix: Optional[str] = None, conv_taps: Optional[int] = None, projection_bias: bool = False,
+                 output_bias: bool = False):
         if num_heads % num_kv_heads:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         if output_gate not in (None, "sigmoid", "sigmoid_head"):
@@ -93,8 +102,21 @@ class GQAAttention(Mixer):
         self.key_dim = head_dim                              # the checkpoint's sizes
         self.value_dim = value_dim if value_dim is not None else head_dim
         self.head_dim = max(self.key_dim, self.value_dim)    # what the cache and the kernels see
+        self.value_blocks = 1                                # ... and blocks of so many value channels per kv head
+        self.conv_taps, self.projection_bias, self.has_output_bias = 1 if conv_taps is None else int(conv_taps), bool(projection_bias), bool(output_bias)
+        self.has_conv = conv_taps is not None
+        self.convolved = bool(self.has_conv or projection_bias)
+        if self.convolved:
+            if tied_values or distance_slopes is not None or qk_norm_eps is not None or head_mixing or value_mix or qk_bias or output_gate == "sigmoid_head":
+                raise ValueError("a convolution of q, k and v or biases of their projections go without tied values, a distance bias, a "
+                                 "q/k norm, mixed heads, shared values and a gate per head")
+            if self.conv_taps < 1:
+                raise ValueError("conv_taps must be positive")
+            self.head_dim, self.value_blocks = ops.value_block_size(self.key_dim, self.value_dim)
         self.q_width = num_heads * self.head_dim
         self.kv_width = num_kv_heads * self.head_dim
+        self.v_width = self.kv_width * self.value_blocks
+        self.o_width = self.q_width * self.value_blocks      # the joined heads
         self.output_gate = output_gate
         self.tied_values = bool(tied_values)
         self.qk_bias = bool(qk_bias)
@@ -112,8 +134,11 @@ class GQAAttention(Mixer):
             raise ValueError(f"unknown value_mix {value_mix!r}")
         self.softcap = None if not softcap else float(softcap)
         self.sink, self.head_mixing, self.value_mix = bool(sink), bool(head_mixing), value_mix
-        self.per_head = bool(self.softcap or self.sink or self.head_mixing or value_mix or output_gate == "sigmoid_head"
-                             or getattr(self.pos, "row_permutation", None) is not None)
+        self.per_head = not self.convolved and bool(self.softcap or self.sink or self.head_mixing or value_mix or output_gate == "sigmoid_head"
+                                                    or getattr(self.pos, "row_permutation", None) is not None)
+        if self.convolved and self.pos is not None and (self.pos.half_split_rotation() is None or not hasattr(self.pos, "angle_table")
+                                                        or self.pos.magnitude != 1.0):
+            raise ValueError("with a convolution of q, k and v the rotation is a half-split one without a magnitude ('rope_scaled')")
         if self.per_head and (self.tied_values or self.distance_slopes is not None or window or qk_norm_eps is not None):
             raise ValueError("bent scores, sinks, mixed heads, shared values and a gate per head go without a window, a distance "
                              "bias, a q/k norm or tied values")
@@ -127,18 +152,28 @@ class GQAAttention(Mixer):
         self.sinks = self.head_mix = self.mix_lambda = None
         # the step takes the route of separate operations (one stacked product, norm and cache write, attention, gate,
         # output product) when any of the options above is on
-        self.extended = bool(output_gate or self.distance_slopes is not None or self.value_dim != self.key_dim or self.tied_values
+        self.extended = bool(self.convolved or output_gate or self.distance_slopes is not None or self.value_dim != self.key_dim or self.tied_values
                              or self.per_head)
-        self.inner_width = self.q_width
-        self.input_width = (self.q_width + (1 if self.tied_values else 2) * self.kv_width
-                            + (self.gate_width if output_gate == "sigmoid_head" else self.q_width if output_gate else 0))
+        self.inner_width = self.o_width
+        self.input_width = (self.q_width + self.kv_width + (0 if self.tied_values else self.v_width)
+                            + (self.gate_width if output_gate == "sigmoid_head" else self.o_width if output_gate else 0))
+        self.in_bias = self.w_conv = self.b_o = None
         self.w_qkv = self.w_o = self.q_norm_w = self.k_norm_w = self.slopes = self.q_bias = self.k_bias = None
 
     def cache_spec(self):
-        return PagedKVSpec(self.num_kv_heads, self.head_dim, self.window)
+        return PagedKVSpec(self.num_kv_heads, self.head_dim, self.window, planes=1 + self.value_blocks)
+
+    def cache_specs(self):
+        # behind the pages: the last taps - 1 projected rows of q, k and v
+        specs = [self.cache_spec()]
+        if self.conv_taps > 1:
+            specs.append(FixedStateSpec((self.conv_taps - 1, self.q_width + self.kv_width + self.v_width), torch.float32))
+        return specs
 
     def attention_geometry(self):
         geo = (self.num_heads, self.num_kv_heads, self.head_dim, self.window or 0)
+        if self.value_blocks > 1:
+            return geo + (False, 1 + self.value_blocks)
         return geo + (True,) if self.distance_slopes is not None else geo
 
     def weight_specs(self, prefix: str) -> list[WeightSpec]:
@@ -164,6 +199,15 @@ class GQAAttention(Mixer):
         if self.qk_bias:
             specs += [WeightSpec(prefix + n["q_bias"], (H * self.key_dim,), VECTOR),
                       WeightSpec(prefix + n["k_bias"], (G * self.key_dim,), VECTOR)]
+        if self.projection_bias:
+            specs += [WeightSpec(prefix + n["q_bias"], (H * self.key_dim,), VECTOR), WeightSpec(prefix + n["k_bias"], (G * self.key_dim,), VECTOR),
+                      WeightSpec(prefix + n["v_bias"], (G * self.value_dim,), VECTOR)]
+        if self.convolved and self.has_conv:
+            specs += [WeightSpec(prefix + n["q_conv"], (H * self.key_dim, self.conv_taps), MATRIX),
+                      WeightSpec(prefix + n["k_conv"], (G * self.key_dim, self.conv_taps), MATRIX),
+                      WeightSpec(prefix + n["v_conv"], (G * self.value_dim, self.conv_taps), MATRIX)]
+        if self.has_output_bias:
+            specs.append(WeightSpec(prefix + n["out_bias"], (W,), VECTOR))
         if self.qk_norm_eps is not None and not self.tied_values:
             specs += [WeightSpec(prefix + n["q_norm"], (self.key_dim,), NORM),
                       WeightSpec(prefix + n["k_norm"], (self.key_dim,), NORM)]
@@ -184,12 +228,12 @@ class GQAAttention(Mixer):
 
         rows = [qk_rows(n["q"], H), qk_rows(n["k"], G)]
         if not self.tied_values:
-            rows.append(_pad_rows(source.get(prefix + n["v"]), G, self.value_dim, D))
+            rows.append(_pad_rows(source.get(prefix + n["v"]), G, self.value_dim, D * self.value_blocks))
         if self.output_gate == "sigmoid_head":
             w_g = source.get(prefix + n["gate"])
             rows.append(torch.cat([w_g, w_g.new_zeros((self.gate_width - H, w_g.shape[1]))], dim=0))
         elif self.output_gate:
-            rows.append(_pad_rows(source.get(prefix + n["gate"]), H, self.value_dim, D))
+            rows.append(_pad_rows(source.get(prefix + n["gate"]), H, self.value_dim, D * self.value_blocks))
         if self.sink:
             self.sinks = source.get(prefix + n["sink"]).to(torch.float32).to(device).contiguous()
         if self.head_mixing:
@@ -198,9 +242,22 @@ class GQAAttention(Mixer):
             self.mix_lambda = float(source.get(prefix + n["value_mix"]).to(torch.float32))
         self.w_qkv = ops.prepare_matrix(torch.cat(rows, dim=0).to(dtype).to(device))
         w_o = source.get(prefix + n["out"])
-        if self.value_dim != D:                      # zero columns where the attention's output is padding
-            w_o = _pad_rows(w_o.t().contiguous(), H, self.value_dim, D).t()
+        if self.value_dim != D * self.value_blocks:  # zero columns where the attention's output is padding
+            w_o = _pad_rows(w_o.t().contiguous(), H, self.value_dim, D * self.value_blocks).t()
         self.w_o = ops.prepare_matrix(w_o.to(dtype).to(device))
+        if self.convolved:
+            # per channel of the stacked q, k and v: the projections' biases, and the taps ([taps, channels])
+            sizes = (("q", H, self.key_dim, D), ("k", G, self.key_dim, D), ("v", G, self.value_dim, D * self.value_blocks))
+
+            def stacked(suffix):
+                return torch.cat([_pad_rows(source.get(prefix + n[x + suffix]).to(torch.float32).reshape(h * d, -1), h, d, pad)
+                                  for x, h, d, pad in sizes], dim=0)
+            if self.projection_bias:
+                self.in_bias = stacked("_bias").reshape(-1).to(device).contiguous()
+            if self.has_conv:
+                self.w_conv = stacked("_conv").t().contiguous().to(device)
+        if self.has_output_bias:
+            self.b_o = source.get(prefix + n["out_bias"]).to(torch.float32).to(device).contiguous()
         if self.qk_bias:
             self.q_bias = source.get(prefix + n["q_bias"]).to(torch.float32).to(device).contiguous()
             self.k_bias = source.get(prefix + n["k_bias"]).to(torch.float32).to(device).contiguous()
@@ -220,6 +277,9 @@ class GQAAttention(Mixer):
     def output_weight(self):
         return self.w_o
 
+    def output_bias(self):
+        return self.b_o
+
     def input_weight(self):
         return self.w_qkv
 
@@ -232,6 +292,9 @@ class GQAAttention(Mixer):
     def mix_projected(self, ctx: StepContext, proj, cache, group, inner, write_cache: bool = True, scale: float = 1.0) -> None:
         T = ctx.num_tokens
         H, Hkv, D = self.num_heads, self.num_kv_heads, self.head_dim
+        if self.convolved:
+            self._mix_convolved(ctx, proj, cache, group, inner, write_cache, scale)
+            return
         view = ctx.groups[group]
         if self.tied_values:
             # q and k lead the rows; the cache's value plane gets the keys as projected, its key plane the normed ones
@@ -267,6 +330,26 @@ class GQAAttention(Mixer):
         if attn is not inner:
             ops.head_norm_gate(attn, proj[:, n_qkv:n_qkv + self.q_width] if self.output_gate else None, None, 0.0, inner, H, D,
                                gate_kind=self.output_gate, scale=scale)
+
+    def _mix_convolved(self, ctx: StepContext, proj, cache, group, inner, write_cache: bool, scale: float) -> None:
+        """Bias, convolution, rotation and cache write in one kernel, attention, the gate per channel."""
+        T = ctx.num_tokens
+        H, Hkv, D, n = self.num_heads, self.num_kv_heads, self.head_dim, self.value_blocks
+        pages, state = cache if isinstance(cache, tuple) else (cache, None)
+        view = ctx.groups[group[0] if isinstance(group, tuple) else group]
+        n_qkv = self.q_width + self.kv_width + self.v_width
+        q = ctx.arena.alloc((T, self.q_width), ctx.dtype)
+        rot = self.pos
+        ops.conv_qkv(proj[:, :n_qkv], self.w_conv, state, ctx, q, pages, view.slot_mapping, H, Hkv, D, in_bias=self.in_bias,
+                     inv_freq=rot.inv_freq if rot is not None else None, rotary_dim=rot.rotary_dim if rot is not None else 0,
+                     cos_sin=rot.angle_table(ctx) if rot is not None else None, write_kv=write_cache)
+        gate = proj[:, n_qkv:n_qkv + self.o_width] if self.output_gate else None
+        direct = gate is None and scale == 1.0 and inner.is_contiguous()
+        attn = inner if direct else ctx.arena.alloc((T, self.o_width), ctx.dtype)
+        ops.paged_attention(q, pages, view.block_tables, ctx, attn, self.scale, self.window or 0, H, Hkv, D, softcap=self.softcap or 0.0,
+                            sinks=self.sinks)
+        if not direct:
+            ops.head_norm_gate(attn, gate, None, 0.0, inner, H, n * D, gate_kind=self.output_gate, scale=scale)
 
     def _mix_per_head(self, ctx: StepContext, proj, qkv, cache, view, inner, write_cache: bool, scale: float) -> None:
         """Rotation (inside the kernel that blends and writes the cache), attention with bent scores or a sink, the heads'

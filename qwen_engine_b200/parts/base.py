@@ -285,6 +285,11 @@ class Mixer(Part):
     inner_width: Optional[int] = None
     input_width: Optional[int] = None
 
+    def output_bias(self) -> Optional[torch.Tensor]:
+        """A bias [hidden] (float32, on the device) that the mixer's result carries and its forward leaves out: the
+        arrangement adds it where the stream is written anyway (an arrangement that cannot refuses the mixer)."""
+        return None
+
     def output_weight(self) -> torch.Tensor:
         raise NotImplementedError
 
@@ -316,6 +321,8 @@ class FeedForward(Part):
 class Block(Part):
     mixer: Mixer
     capturable = True             # False if any of its parts says so: steps of the model are then never graph-captured
+    adds_output_bias = False      # True if the block adds its mixer's output_bias() to the stream
+    takes_second = False          # True if the block's first norm adds both of two pending branch outputs (ops.ResidualStream.second)
     keeps_copy = False            # True if the block reads the stream's rounded copy and leaves it up to date (ops.ResidualStream.copy)
 
     def cache_specs(self) -> list:

@@ -53,6 +53,19 @@ class RMSNorm(Norm):
         ops.add_rmsnorm(resid, delta, self.weight, self.eps, out)
         return out
 
+    def normed_pair(self, ctx: StepContext, stream, other: "RMSNorm | None", bias=None):
+        """This norm's and ``other``'s rows of the stream after its pending branch outputs are added, from one pass over the
+        stream (``other`` None: this norm's alone); ``bias`` joins the stream behind the norms."""
+        if other is not None and (other.width, other.eps) != (self.width, self.eps):
+            raise ValueError("rmsnorm: two norms of one pass have one width and one eps")
+        out = [ctx.arena.alloc(tuple(stream.resid.shape), ctx.dtype) for _ in range(1 if other is None else 2)]
+        ops.add_rmsnorm_pair(stream.resid, stream.delta if stream.has_delta else None, stream.second if stream.has_second else None,
+                             bias, self.weight, out[0], None if other is None else other.weight, None if other is None else out[1],
+                             self.eps)
+        stream.has_delta = stream.has_second = False
+        stream.n_ssq = 0
+        return out[0], (None if other is None else out[1])
+
     def add_norm_rows(self, ctx: StepContext, resid, delta, rows, out):
         ops.add_rmsnorm_rows(resid, delta, rows, self.weight, self.eps, out)
         return out

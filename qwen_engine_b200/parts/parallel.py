@@ -39,6 +39,7 @@ class ParallelMixers(Mixer):
         self.joined = all(b.inner_width is not None for b in self.branches)
         self.inner_width = sum(b.inner_width for b in self.branches) if self.joined else None
         self.w_o: Optional[torch.Tensor] = None
+        self.b_o: Optional[torch.Tensor] = None       # the branches' output biases, weighted and summed (where any has one)
         self.w_in: Optional[torch.Tensor] = None      # the branches' stacked input weights, stacked once more (if all offer them)
         self._n_caches = [len(b.cache_specs()) for b in self.branches]
 
@@ -58,6 +59,8 @@ class ParallelMixers(Mixer):
     def load(self, prefix, source, dtype, device) -> None:
         for b, p in zip(self.branches, self.prefixes):
             b.load(prefix + p, source, dtype, device)
+        biases = [(b.output_bias(), s) for b, s in zip(self.branches, self.scales) if b.output_bias() is not None]
+        self.b_o = sum(s * b for b, s in biases) if biases else None
         if self.joined:
             # [hidden, inner_1 + inner_2 + ...]: the sum over branches happens inside the product
             self.w_o = ops.prepare_matrix(torch.cat([b.output_weight() for b in self.branches], dim=1))
@@ -71,6 +74,9 @@ class ParallelMixers(Mixer):
 
     def output_weight(self):
         return self.w_o
+
+    def output_bias(self):
+        return self.b_o
 
     def _caches(self, cache, group):
         """The branches' shares of the tuples of caches and groups the plan handed over."""

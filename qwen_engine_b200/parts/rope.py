@@ -87,7 +87,7 @@ def ramped_frequencies(inv_freq: torch.Tensor, base: float, rotary_dim: int, fac
 class ScaledRope(NeoxRope):
     """Rotation of the first ``rotary_dim`` channels of a head with scaled frequencies.
 
-    ``scaling``: None, or ("bands", factor, low, high, original) (``banded_frequencies``), or ("ramp", factor, original,
+    ``scaling``: None, or ("linear", factor) (every frequency divided by it), or ("bands", factor, low, high, original) (``banded_frequencies``), or ("ramp", factor, original,
     fast, slow) (``ramped_frequencies``, with which cosines and sines are also multiplied by 0.1 ln(factor) + 1).
     ``pairing``: "half" pairs channel i with i + rotary_dim / 2; "interleaved" pairs 2 i with 2 i + 1.  The kernels
     rotate half-split pairs; for interleaved pairs the mixer reorders the rows of W_q and W_k within every head when it
@@ -103,6 +103,8 @@ class ScaledRope(NeoxRope):
         base = torch.tensor([self.theta ** (-2.0 * i / self.rotary_dim) for i in range(self.rotary_dim // 2)], dtype=torch.float64)
         if self.scaling is None:
             f = base
+        elif self.scaling[0] == "linear":
+            f = base / float(self.scaling[1])
         elif self.scaling[0] == "bands":
             _, factor, low, high, original = self.scaling
             f = banded_frequencies(base, float(factor), float(low), float(high), original)
@@ -116,6 +118,20 @@ class ScaledRope(NeoxRope):
 
     def step_table(self, ctx: StepContext):
         return None           # (the table of a step's angles serves whole heads of 128 channels without a magnitude)
+
+    def angle_table(self, ctx: StepContext):
+        """The cosines and sines of this step's angles [T, rotary_dim / 2, 2] for the kernels that take a table for any
+        number of rotated channels (``ops.conv_qkv``), formed once per step for all layers with the same frequencies; None
+        for steps of few tokens (the kernel then computes the angles itself)."""
+        if ctx.num_tokens < ops.ROPE_TABLE_MIN_T or self.magnitude != 1.0:
+            return None
+        key = ("angle_table", self.theta, self.rotary_dim, self.scaling)
+        table = ctx.extras.get(key)
+        if table is None:
+            table = ctx.arena.alloc_step((ctx.num_tokens, self.rotary_dim // 2, 2), torch.float32)
+            ops.rope_table(ctx.positions, self.inv_freq, table)
+            ctx.extras[key] = table
+        return table
 
     def row_permutation(self):
         """None, or the order in which a head's rows of W_q and W_k are to be stacked so that the kernels' half-split

@@ -11,9 +11,10 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Callable
 
-from .config import BesavikConfig, ConfigError, GanidraConfig, MerudraConfig, ModelConfig, PufivikConfig, Qwen3Config, ZugunexConfig, read_config_json
+from .config import BesavikConfig, ConfigError, FunudraConfig, GanidraConfig, MerudraConfig, ModelConfig, PufivikConfig, Qwen3Config, ZugunexConfig, read_config_json
 from .models.decoder import DecoderModel, ModelLayout
 from .models.besavik import besavik_layout
+from .models.funudra import funudra_layout
 from .models.ganidra import ganidra_layout
 from .models.merudra import merudra_layout
 from .models.pufivik import pufivik_layout
@@ -41,6 +42,7 @@ register_architecture("Besavik", BesavikConfig, besavik_layout)
 register_architecture("Merudra", MerudraConfig, merudra_layout)
 register_architecture("Pufivik", PufivikConfig, pufivik_layout)
 register_architecture("Zugunex", ZugunexConfig, zugunex_layout)
+register_architecture("Funudra", FunudraConfig, funudra_layout)
 
 
 def architecture_of(raw_config: dict[str, Any]) -> Architecture:

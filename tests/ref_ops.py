@@ -157,6 +157,14 @@ def paged_attention(qkv, kv_pages, block_tables, ctx, out, scale, window, num_he
     softmax(scale q k^T + mask) v with key j allowed for the query at position i iff
     j <= i and (window == 0 or j > i - window)."""
     Hq, Hkv, D = num_heads, num_kv_heads, head_dim
+    if kv_pages.shape[1] > 2:             # n blocks of D value channels: out [T, Hq n D], one block after the other
+        n = kv_pages.shape[1] - 1
+        part = torch.zeros(out.shape[0], num_heads * head_dim, dtype=out.dtype)
+        for b in range(n):
+            paged_attention(qkv, kv_pages[:, [0, 1 + b]], block_tables, ctx, part, scale, window, num_heads, num_kv_heads, head_dim, None, None,
+                            softcap, sinks)
+            out.view(out.shape[0], num_heads, n, head_dim)[:, :, b] = part.view(out.shape[0], num_heads, head_dim)
+        return
     if value_shifts > 1:                  # out [S, T, Hq D]: one output per shift of the values' kv head
         for s in range(value_shifts):
             paged_attention(qkv, kv_pages, block_tables, ctx, out[s], scale, window, Hq, Hkv, D, next_pages, slopes, softcap, sinks, s)
@@ -546,6 +554,131 @@ def linear_silu_mul(gate_up, w, out, scratch):
     linear(act, w, out)
 
 
+def add_rmsnorm_pair(resid, delta_a, delta_b, bias, w1, out1, w2, out2, eps):
+    for d in (delta_a, delta_b):
+        if d is not None:
+            resid.add_(d.to(torch.float32))
+    out1.copy_(_rms(resid, w1, eps).to(out1.dtype))
+    if out2 is not None:
+        out2.copy_(_rms(resid, w2, eps).to(out2.dtype))
+    if bias is not None:
+        resid.add_(bias)
+
+
+def group_norm_gate(x, gate, weight, eps, groups, out, gate_kind="silu", gate_first=False, divisor=None, scale=1.0):
+    T, C = x.shape
+    y = x.to(torch.float32).reshape(T, groups, C // groups)
+    if divisor is not None:
+        y = y / divisor[:, :, None]
+    g = None
+    if gate is not None:
+        g = gate.to(torch.float32).reshape(T, groups, C // groups)
+        g = g * torch.sigmoid(g) if gate_kind == "silu" else torch.sigmoid(g)
+    if g is not None and gate_first:
+        y = y * g
+    y = y / torch.sqrt((y * y).mean(dim=-1, keepdim=True) + eps) * weight.reshape(groups, C // groups)
+    if g is not None and not gate_first:
+        y = y * g
+    out.copy_((y * scale).reshape(T, C).to(out.dtype))
+
+
+def _conv_rows(x, w, state, ctx, in_bias, write_state):
+    """float32 [T, C]: the convolution's rows, the state moved on."""
+    T, C = x.shape
+    taps = 1 if w is None else w.shape[0]
+    u = x.to(torch.float32)
+    if in_bias is not None:
+        u = u + in_bias
+    if w is None:
+        return u
+    hist = taps - 1
+    y = torch.zeros(T, C, dtype=torch.float32)
+    cu, ctx_lens, slots = ctx.cu_q.tolist(), ctx.ctx_lens.tolist(), ctx.slot_ids.tolist()
+    for r in range(len(ctx_lens)):
+        a, b = cu[r], cu[r + 1]
+        if b <= a:
+            continue
+        old = state[slots[r]].clone() if hist and ctx_lens[r] > 0 else torch.zeros(hist, C)
+        seq = torch.cat([old, u[a:b]], dim=0)
+        for j in range(taps):
+            y[a:b] += seq[j:j + b - a] * w[j][None, :]
+        if write_state and hist:
+            state[slots[r]] = seq[-hist:]
+    return y
+
+
+def conv_act(x, w, state, ctx, out, in_bias=None, out_bias=None, silu=True, write_state=True):
+    y = _conv_rows(x, w, state, ctx, in_bias, write_state)
+    if out_bias is not None:
+        y = y + out_bias
+    out.copy_((y * torch.sigmoid(y) if silu else y).to(out.dtype))
+
+
+def conv_qkv(x, w, state, ctx, q, kv_pages, slot_mapping, num_heads, num_kv_heads, head_dim, in_bias=None, inv_freq=None, rotary_dim=0,
+             cos_sin=None, write_kv=True):
+    T = x.shape[0]
+    Hq, Hkv, D = num_heads, num_kv_heads, head_dim
+    n = kv_pages.shape[1] - 1
+    y = _conv_rows(x, w, state, ctx, in_bias, write_kv)
+    qq = y[:, :Hq * D].reshape(T, Hq, D)
+    k = y[:, Hq * D:(Hq + Hkv) * D].reshape(T, Hkv, D)
+    v = y[:, (Hq + Hkv) * D:].reshape(T, Hkv, n, D)
+    if inv_freq is not None:
+        qq = _rotate(qq, ctx.positions, inv_freq, rotary_dim)
+        k = _rotate(k, ctx.positions, inv_freq, rotary_dim)
+    q.copy_(qq.reshape(T, Hq * D).to(q.dtype))
+    if write_kv:
+        P = kv_pages.shape[3]
+        slots = slot_mapping.long()
+        page, off = slots // P, slots % P
+        kv_pages[page, 0, :, off, :] = k.to(kv_pages.dtype)
+        for i in range(n):
+            kv_pages[page, 1 + i, :, off, :] = v[:, :, i].to(kv_pages.dtype)
+
+
+def state_space_scan(x, B, C, dt, dt_bias, log_rate, skip, state, ctx, out, num_heads, num_groups, state_dim, value_dim, write_state=True):
+    H, G, N, P = num_heads, num_groups, state_dim, value_dim
+    d = torch.nn.functional.softplus(dt.to(torch.float32) + (0.0 if dt_bias is None else dt_bias), threshold=50.0)      # [T, H]
+    a = torch.exp(-torch.exp(log_rate) * d)
+    cu, ctx_lens, slots = ctx.cu_q.tolist(), ctx.ctx_lens.tolist(), ctx.slot_ids.tolist()
+    for r in range(len(ctx_lens)):
+        S = state[slots[r]].clone() if ctx_lens[r] > 0 else torch.zeros_like(state[slots[r]])       # [H, P, N]
+        for t in range(cu[r], cu[r + 1]):
+            Bt = B[t].to(torch.float32).reshape(G, N).repeat_interleave(H // G, dim=0)
+            Ct = C[t].to(torch.float32).reshape(G, N).repeat_interleave(H // G, dim=0)
+            xt = x[t].to(torch.float32).reshape(H, P)
+            S = a[t][:, None, None] * S + (d[t][:, None] * xt)[:, :, None] * Bt[:, None, :]
+            y = (S * Ct[:, None, :]).sum(dim=-1)
+            if skip is not None:
+                y = y + skip[:, None] * xt
+            out[t] = y.reshape(H * P)
+        if write_state and cu[r + 1] > cu[r]:
+            state[slots[r]] = S
+
+
+def matrix_memory_scan(q, k, v, gate_in, gate_keep, bias_in, bias_keep, cap, state, maxima, ctx, out, divisor, q_scale, den_eps, num_heads,
+                       key_dim, value_dim, write_state=True):
+    H, dk, dv = num_heads, key_dim, value_dim
+    gi = cap * torch.tanh((gate_in.to(torch.float32) + (0.0 if bias_in is None else bias_in)) / cap)
+    gf = torch.nn.functional.logsigmoid(cap * torch.tanh((gate_keep.to(torch.float32) + (0.0 if bias_keep is None else bias_keep)) / cap))
+    cu, ctx_lens, slots = ctx.cu_q.tolist(), ctx.ctx_lens.tolist(), ctx.slot_ids.tolist()
+    for r in range(len(ctx_lens)):
+        fresh = ctx_lens[r] == 0
+        S = torch.zeros_like(state[slots[r]]) if fresh else state[slots[r]].clone()                 # [H, dv + 1, dk]
+        m = torch.zeros(H) if fresh else maxima[slots[r], :, 0].clone()
+        for t in range(cu[r], cu[r + 1]):
+            kept = gf[t] + m
+            m = torch.maximum(kept, gi[t])
+            vt = torch.cat([v[t].to(torch.float32).reshape(H, dv), torch.ones(H, 1)], dim=1)
+            S = torch.exp(kept - m)[:, None, None] * S + (torch.exp(gi[t] - m)[:, None] * vt)[:, :, None] * k[t].to(torch.float32).reshape(H, 1, dk)
+            y = (S * (q[t].to(torch.float32).reshape(H, 1, dk) * q_scale)).sum(dim=-1)
+            out[t] = y[:, :dv].reshape(H * dv)
+            divisor[t] = torch.maximum(y[:, dv].abs(), torch.exp(-m)) + den_eps
+        if write_state and cu[r + 1] > cu[r]:
+            state[slots[r]] = S
+            maxima[slots[r]] = m[:, None].expand(H, dv + 1)
+
+
 def argmax(logits, out):
     out.copy_(torch.argmax(logits, dim=-1).to(torch.int32))
 
@@ -591,7 +724,7 @@ def copy_pages(cache, pairs):
         cache[:, dst] = cache[:, src].clone()
 
 
-_NAMES = ["group_rmsnorm", "group_norm_add", "head_mix_gate", "qk_bias_norm_kv_write", "stream_conv", "gated_norm_add", "token_side_gate", "depth_mix", "latent_prepare", "head_linear", "short_conv", "unit_norm", "delta_rule_scan", "moe_route", "moe_experts",
+_NAMES = ["add_rmsnorm_pair", "group_norm_gate", "conv_act", "conv_qkv", "state_space_scan", "matrix_memory_scan", "group_rmsnorm", "group_norm_add", "head_mix_gate", "qk_bias_norm_kv_write", "stream_conv", "gated_norm_add", "token_side_gate", "depth_mix", "latent_prepare", "head_linear", "short_conv", "unit_norm", "delta_rule_scan", "moe_route", "moe_experts",
           "act_mul", "channel_decay", "linear_attention_scan", "head_norm_gate", "scaled_add", "copy_pages", "swiglu_small_applies", "qkv_rope_small_applies", "prepare_matrix", "embedding", "add_rmsnorm", "add_rmsnorm_rows", "linear",
           "qk_norm_rope_kv_write", "rope_neox", "rope_table", "place_tokens", "swiglu_fused_applies", "plan_attention", "paged_attention", "silu_mul", "linear_silu_mul",
           "argmax", "sample"]
