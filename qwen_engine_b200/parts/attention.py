@@ -55,7 +55,7 @@ import torch
 
 from .. import ops
 from ..cache.spec import FixedStateSpec, PagedKVSpec
-from ..weights.spec import MATRIX, NORM, VECTOR, WeightSpec
+from ..weights.spec import MATRIX, NORM, TAPS, VECTOR, WeightSpec
 from .base import Mixer, PartSpec, StepContext, register, step_hint
 
 _NAMES = dict(q="q_proj.weight", k="k_proj.weight", v="v_proj.weight", out="o_proj.weight",
@@ -203,9 +203,9 @@ class GQAAttention(Mixer):
             specs += [WeightSpec(prefix + n["q_bias"], (H * self.key_dim,), VECTOR), WeightSpec(prefix + n["k_bias"], (G * self.key_dim,), VECTOR),
                       WeightSpec(prefix + n["v_bias"], (G * self.value_dim,), VECTOR)]
         if self.convolved and self.has_conv:
-            specs += [WeightSpec(prefix + n["q_conv"], (H * self.key_dim, self.conv_taps), MATRIX),
-                      WeightSpec(prefix + n["k_conv"], (G * self.key_dim, self.conv_taps), MATRIX),
-                      WeightSpec(prefix + n["v_conv"], (G * self.value_dim, self.conv_taps), MATRIX)]
+            specs += [WeightSpec(prefix + n["q_conv"], (H * self.key_dim, self.conv_taps), TAPS),
+                      WeightSpec(prefix + n["k_conv"], (G * self.key_dim, self.conv_taps), TAPS),
+                      WeightSpec(prefix + n["v_conv"], (G * self.value_dim, self.conv_taps), TAPS)]
         if self.has_output_bias:
             specs.append(WeightSpec(prefix + n["out_bias"], (W,), VECTOR))
         if self.qk_norm_eps is not None and not self.tied_values:

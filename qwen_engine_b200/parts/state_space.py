@@ -22,7 +22,7 @@ import torch
 
 from .. import ops
 from ..cache.spec import FixedStateSpec
-from ..weights.spec import MATRIX, NORM, VECTOR, WeightSpec
+from ..weights.spec import MATRIX, NORM, TAPS, VECTOR, WeightSpec
 from .base import Mixer, StepContext, register
 
 _NAMES = {"in": "in", "conv": "conv", "conv_bias": "conv.b", "dt_bias": "dt_bias", "rate": "A_log", "skip": "D", "norm": "norm", "out": "o"}
@@ -62,7 +62,7 @@ class StateSpace(Mixer):
     def weight_specs(self, prefix: str) -> list[WeightSpec]:
         n, W, H = self.names, self.hidden_size, self.num_heads
         return [WeightSpec(prefix + n["in"], (self.stored_width, W), MATRIX),
-                WeightSpec(prefix + n["conv"], (self.conv_width, self.conv_taps), MATRIX),
+                WeightSpec(prefix + n["conv"], (self.conv_width, self.conv_taps), TAPS),
                 WeightSpec(prefix + n["conv_bias"], (self.conv_width,), VECTOR),
                 WeightSpec(prefix + n["dt_bias"], (H,), VECTOR),
                 WeightSpec(prefix + n["rate"], (H,), VECTOR),

@@ -16,7 +16,7 @@ import torch
 from safetensors.torch import save_file
 
 from ..config import ModelConfig, write_config_json
-from .spec import MATRIX, NORM, NORM_ZERO, VECTOR, WeightSpec
+from .spec import MATRIX, NORM, NORM_ZERO, TAPS, VECTOR, WeightSpec
 
 
 def _tensor_seed(seed: int, name: str) -> int:
@@ -28,7 +28,7 @@ class RandomSource:
     """A TensorSource that makes each tensor when asked.
 
     Matrices are N(0, std); norm scales are 1 + N(0, norm_std), or N(0, norm_std) where the norm
-    adds the one itself; biases are N(0, 1).  Values are drawn
+    adds the one itself; biases are N(0, 1), a convolution's n taps N(0, 1 / n).  Values are drawn
     in float32 on the CPU and rounded to ``store_dtype``."""
 
     def __init__(self, manifest: Iterable[WeightSpec], seed: int, std: float = 0.02,
@@ -53,6 +53,8 @@ class RandomSource:
             t = self.norm_std * t
         elif spec.kind == VECTOR:
             pass                                     # a bias: N(0, 1), so that what it feeds (a decay) varies
+        elif spec.kind == TAPS:
+            t = t * spec.drawn_shape[-1] ** -0.5     # so that what passes the convolution keeps its size
         elif spec.kind == MATRIX:
             t = self.std * t
         else:

@@ -11,6 +11,7 @@ MATRIX = "matrix"        # [out, in] projection or embedding table: compute dtyp
 NORM = "norm"            # scale vector of a norm: always float32 on the device
 NORM_ZERO = "norm_zero"  # scale vector of a norm that is stored around zero (the norm multiplies by 1 + w): float32
 VECTOR = "vector"        # a bias: float32 on the device
+TAPS = "taps"            # [channels, taps] of a convolution over time on each channel: float32 on the device
 
 
 @dataclass(frozen=True)

@@ -60,14 +60,12 @@ def rotation_frequencies(base, dims, factor):
 
 def rotate_half_split(x, dims, freqs):
     """x [T, D]: the pairs (i, i + dims/2) of the first ``dims`` channels turn by position * freqs[i]."""
-    T, half = x.shape[0], dims // 2
+    half = dims // 2
+    a = torch.arange(x.shape[0], dtype=x.dtype)[:, None] * torch.tensor(freqs, dtype=x.dtype)[None, :]
     out = x.clone()
-    for p in range(T):
-        for i in range(half):
-            a = p * freqs[i]
-            u, v = x[p, i], x[p, i + half]
-            out[p, i] = u * math.cos(a) - v * math.sin(a)
-            out[p, i + half] = v * math.cos(a) + u * math.sin(a)
+    u, v = x[:, :half], x[:, half:dims]
+    out[:, :half] = u * torch.cos(a) - v * torch.sin(a)
+    out[:, half:dims] = v * torch.cos(a) + u * torch.sin(a)
     return out
 
 
