@@ -463,7 +463,8 @@ _TIMED_OPS = ("embedding", "linear", "linear_swiglu", "linear_swiglu_small", "li
               "qk_norm_rope_kv_write", "paged_attention", "channel_decay", "linear_attention_scan", "head_norm_gate",
               "add_rmsnorm", "add_rmsnorm_rows", "rope_table", "latent_prepare", "head_linear", "short_conv", "unit_norm",
               "delta_rule_scan", "moe_route", "moe_experts", "qk_bias_norm_kv_write", "stream_conv", "gated_norm_add",
-              "token_side_gate", "depth_mix", "group_rmsnorm", "group_norm_add", "head_mix_gate")
+              "token_side_gate", "depth_mix", "group_rmsnorm", "group_norm_add", "head_mix_gate", "add_rmsnorm_pair", "group_norm_gate",
+              "conv_act", "conv_qkv", "state_space_scan", "matrix_memory_scan")
 
 
 def ganidra_config_of(sz: dict) -> dict:
@@ -540,6 +541,158 @@ def zugunex_config_of(sz: dict) -> dict:
     layers = [dict(type="latent_attention", mixer=own if i % 2 == 0 else dict(own, kv_from=i - 1), mlp=dense if i == 0 else moe)
               for i in range(sz["layers"])]
     return dict(architecture="Zugunex", vocab=sz["vocab"], width=sz["width"], norm=dict(eps=1e-6), layers=layers)
+
+
+def funudra_config_of(sz: dict) -> dict:
+    """A Funudra model at the sizes of ``sz``: state-space layers (twice the width, heads of 64 channels, 128 state channels,
+    eight groups) and layers of softmax attention (values of twice the keys' size, half of every head rotated,
+    convolutions of four taps, bent scores) beside a matrix memory (half of the linear attention's heads, its key and value
+    sizes), in turn; a dense feed-forward without a gate beside every mixer."""
+    D, ssm_heads = sz["head_dim"], 2 * sz["width"] // 64
+    ssm = dict(heads=ssm_heads, vdim=64, state=128, groups=8, conv=4, norm_groups=8)
+    left = dict(heads=sz["heads"], kv_heads=sz["kv_heads"], dim=D, vdim=2 * D, conv=4, scale=D ** -0.5, softcap=50.0,
+                rot=dict(base=500000.0, dims=D // 2, scaling=dict(factor=4.0)))
+    right = dict(heads=max(1, sz["gla_heads"] // 2), dim=sz["gla_dk"], vdim=sz["gla_dv"], gate_cap=15.0)
+    mlp = dict(kind="dense", ff=sz["ff"])
+    pair = [dict(type="mamba2", mixer=ssm, mlp=mlp),
+            dict(type="parallel", mixer=dict(left=left, right=right, left_scale=0.7, right_scale=0.7), mlp=mlp)]
+    return dict(architecture="Funudra", vocab=sz["vocab"], width=sz["width"], norm=dict(eps=1e-6), layers=pair * (sz["layers"] // 2))
+
+
+def funudra_kernels_alone(torch, ops, peaks) -> dict:
+    """The kernels and kernel options that Funudra adds, each alone beside its like among the other models' kernels: device
+    time (CUDA events around three replays of a graph of ten launches); for passes over rows the bytes moved over the
+    measured copy rate (rows larger than L2), for recurrences also the state's elements updated a microsecond, for
+    attention the multiply-adds over the measured bfloat16 rate, for decoded tokens the bytes over the copy rate."""
+    from types import SimpleNamespace
+    from qwen_engine_b200.engine.runner import ModelRunner
+    from qwen_engine_b200.parts.base import Arena
+    dev, bf, f32 = "cuda:0", torch.bfloat16, torch.float32
+    hbm, tflops = float(peaks["hbm_gbs"]), float(peaks["bf16_tflops"])
+    g = torch.Generator(device=dev).manual_seed(7)
+    rnd = lambda *shape, dtype=f32, std=1.0: (torch.randn(*shape, device=dev, dtype=f32, generator=g) * std).to(dtype)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    out: dict = {}
+
+    def timed(name, fn, nbytes=None, flops=None, like=None, elements=None):
+        for _ in range(3):
+            fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(10):
+                fn()
+        graph.replay()
+        torch.cuda.synchronize()
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        for _ in range(3):
+            graph.replay()
+        b.record()
+        torch.cuda.synchronize()
+        us = a.elapsed_time(b) * 1000.0 / 30.0
+        rec = {"us": round(us, 1)}
+        if nbytes:
+            rec.update(mb=round(nbytes / 1e6, 1), frac_of_copy=round(nbytes / us / 1e3 / hbm, 3))
+        if flops:
+            rec.update(tflops=round(flops / us / 1e6, 1), frac_of_bf16=round(flops / us / 1e6 / tflops, 3))
+        if elements:
+            rec["state_elements_per_us"] = round(elements / us / 1e3) * 1000
+        if like:
+            rec["like"] = like
+        out[name] = rec
+
+    def step(reqs, n, ctx_len):
+        return SimpleNamespace(cu_q=i32([r * n for r in range(reqs + 1)]), ctx_lens=i32([ctx_len] * reqs), slot_ids=i32(list(range(reqs))),
+                               num_reqs=reqs, max_q_len=n, positions=i32([ctx_len + i for _ in range(reqs) for i in range(n)]))
+    T, W, reqs = 16384, 2048, 8
+    stream, da, db = rnd(T, W), rnd(T, W, dtype=bf, std=0.01), rnd(T, W, dtype=bf, std=0.01)
+    o1, o2, w1, w2, bias = torch.empty(T, W, device=dev, dtype=bf), torch.empty(T, W, device=dev, dtype=bf), rnd(W), rnd(W), rnd(W, std=0.01)
+    timed("add_rmsnorm_pair", lambda: ops.add_rmsnorm_pair(stream, da, db, bias, w1, o1, w2, o2, 1e-6), T * W * 16, like="add_rmsnorm")
+    timed("add_rmsnorm", lambda: ops.add_rmsnorm(stream, da, w1, 1e-6, o1), T * W * 12)
+    del stream, da, db, o1, o2
+    ctx = step(reqs, T // reqs, 0)
+    C, taps = 4096 + 2048, 4
+    x, wc, state = rnd(T, C, dtype=bf), rnd(taps, C), torch.zeros(reqs, taps - 1, C, device=dev)
+    xo, xf, wn = torch.empty(T, C, device=dev, dtype=bf), torch.empty(T, C, device=dev), rnd(C, taps)
+    cb = rnd(C)
+    timed("conv_act with bias and silu", lambda: ops.conv_act(x, wc, state, ctx, xo, out_bias=cb, silu=True), T * C * 4, like="short_conv")
+    timed("short_conv", lambda: ops.short_conv(x, wn, state, ctx, xf, silu=True), T * C * 6)
+    del xo, xf
+    Hq, Hkv, D, page = 16, 8, 128, 16
+    slots = torch.arange(T, device=dev, dtype=torch.int32)
+    inv = (1.0 / (1e6 ** (torch.arange(0, D // 2, 2, device=dev, dtype=f32) / (D // 2)))).contiguous()
+    inv_all = (1.0 / (1e6 ** (torch.arange(0, D, 2, device=dev, dtype=f32) / D))).contiguous()
+    table = torch.empty(T, D // 4, 2, device=dev)
+    ops.rope_table(ctx.positions, inv, table)
+    C2 = (Hq + 3 * Hkv) * D
+    proj, wq, st2, q = rnd(T, C2, dtype=bf), rnd(taps, C2), torch.zeros(reqs, taps - 1, C2, device=dev), torch.empty(T, Hq * D, device=dev, dtype=bf)
+    pages3 = rnd(T // page, 3, Hkv, page, D, dtype=bf)
+    b2 = rnd(C2)
+    timed("conv_qkv, two blocks of values", lambda: ops.conv_qkv(proj, wq, st2, ctx, q, pages3, slots, Hq, Hkv, D, in_bias=b2, inv_freq=inv,
+                                                                 rotary_dim=D // 2, cos_sin=table), T * C2 * 4, like="qk_norm_rope_kv_write")
+    pages2, nw, qkv = rnd(T // page, 2, Hkv, page, D, dtype=bf), rnd(D), rnd(T, (Hq + 2 * Hkv) * D, dtype=bf)
+    timed("qk_norm_rope_kv_write", lambda: ops.qk_norm_rope_kv_write(qkv, ctx.positions, nw, nw, 1e-6, inv_all, D, pages2, slots, Hq, Hkv, D),
+          T * ((Hq + 2 * Hkv) * D) * 4)
+    y, gate, res, wg = rnd(T, 4096), rnd(T, 4096, dtype=bf), torch.empty(T, 4096, device=dev, dtype=bf), rnd(4096)
+    timed("group_norm_gate, eight groups of 512, gate first", lambda: ops.group_norm_gate(y, gate, wg, 1e-6, 8, res, gate_first=True), T * 4096 * 8, like="head_norm_gate")
+    div = rnd(T, 32).abs() + 1.0
+    timed("group_norm_gate, heads of 128 with divisors", lambda: ops.group_norm_gate(y, gate, wg, 1e-6, 32, res, gate_kind="sigmoid", divisor=div), T * 4096 * 8, like="head_norm_gate")
+    timed("head_norm_gate, heads of 128", lambda: ops.head_norm_gate(y, gate, wg[:128].contiguous(), 1e-6, res, 32, 128, gate_kind="silu"), T * 4096 * 8)
+    timed("head_norm_gate, one head of 4 096", lambda: ops.head_norm_gate(y, gate, wg, 1e-6, res, 1, 4096, gate_kind="sigmoid"), T * 4096 * 8)
+    del y, gate, res, x, proj, pages3, pages2, qkv
+    # recurrences: one prompt of 2 048 tokens, eight of them, and 64 decoded tokens
+    for label, R, n, c in (("2 048 tokens", 1, 2048, 0), ("8 x 2 048 tokens", 8, 2048, 0), ("64 decoded tokens", 64, 1, 500)):
+        ctx, t = step(R, n, c), R * n
+        for H, G, N, P in ((64, 8, 128, 64),):
+            xs, B, Cc, dt = rnd(t, H * P, dtype=bf), rnd(t, G * N, dtype=bf, std=0.1), rnd(t, G * N, dtype=bf), rnd(t, H, dtype=bf)
+            stt, o = torch.zeros(R, H, P, N, device=dev), torch.empty(t, H * P, device=dev)
+            hb = rnd(H)
+            moved = t * (H * P * 6 + 2 * G * N * 2 + H * 2) + 2 * stt.numel() * 4
+            timed(f"state_space_scan, {H} heads, {N} x {P}, {label}", lambda: ops.state_space_scan(xs, B, Cc, dt, hb, hb, hb, stt, ctx, o, H, G, N, P),
+                  moved, elements=t * H * N * P, like="linear_attention_scan")
+        H, dk, dv = 16, 64, 128
+        q, k, v, al = rnd(t, H * dk, dtype=bf), rnd(t, H * dk, dtype=bf), rnd(t, H * dv, dtype=bf), torch.rand(t, H * dk, device=dev, generator=g)
+        stt, o, hb = torch.zeros(R, H, dv, dk, device=dev), torch.empty(t, H * dv, device=dev), rnd(H)
+        moved = t * (2 * H * dk * 2 + H * dv * 6) + 2 * stt.numel() * 4
+        timed(f"linear_attention_scan, {H} heads, {dk} x {dv}, {label}", lambda: ops.linear_attention_scan(q, k, v, al, stt, ctx, o, 0.125, H, dk, dv),
+              moved + t * H * dk * 4, elements=t * H * dk * dv)
+        sm, mx, gi, gf, dv_ = torch.zeros(R, H, dv + 1, dk, device=dev), torch.zeros(R, H, dv + 1, device=dev), rnd(t, H, dtype=bf), rnd(t, H, dtype=bf), torch.empty(t, H, device=dev)
+        timed(f"matrix_memory_scan, {H} heads, {dk} x {dv}, {label}",
+              lambda: ops.matrix_memory_scan(q, k, v, gi, gf, hb, hb, 15.0, sm, mx, ctx, o, dv_, 0.125, 1e-6, H, dk, dv), moved, elements=t * H * dk * dv,
+              like="linear_attention_scan")
+    # attention with bent scores: keys of 128 and values of 256 channels (two blocks) beside 128 and 128
+    for kind, q_lens, ctx_lens in (("4 x 2 048 tokens", [2048] * 4, [0] * 4), ("2 048 tokens", [2048], [0]), ("8 decoded tokens", [1] * 8, [2047] * 8),
+                                   ("64 decoded tokens", [1] * 64, [2047] * 64)):
+        R, t = len(q_lens), sum(q_lens)
+        blocks = 2048 // page
+        tables = torch.arange(R * blocks, device=dev, dtype=torch.int32).view(R, blocks).contiguous()
+        prompts = q_lens[0] > 1
+        q = rnd(t, Hq * D, dtype=bf)
+        pairs = sum(c + i + 1 for m, c in zip(q_lens, ctx_lens) for i in range(m))
+        for n in (2, 1):
+            pages = rnd(R * blocks, 1 + n, Hkv, page, D, dtype=bf)
+            geo = (Hq, Hkv, D, 0, False, 1 + n) if n > 1 else (Hq, Hkv, D, 0)
+            splits = None if prompts else ops.decode_splits(R, 2048, (geo,), bf)
+            plan = ops.plan_attention(q_lens, ctx_lens, page, (geo,), bf, uniform_splits=splits)
+            devplan = ModelRunner._device_plan(plan, {"plan_" + k_: i32(v_) for k_, v_ in plan.items()}, (geo,))
+            cu = [0]
+            for m in q_lens:
+                cu.append(cu[-1] + m)
+            actx = SimpleNamespace(cu_q=i32(cu), ctx_lens=i32(ctx_lens), q_lens_host=q_lens, ctx_lens_host=ctx_lens, attn_plan=devplan,
+                                   max_q_len=max(q_lens), arena=Arena(dev, 1 << 28))
+            res = torch.empty(t, Hq * n * D, device=dev, dtype=bf)
+
+            def attend():
+                m = actx.arena.mark()
+                ops.paged_attention(q, pages, tables, actx, res, D ** -0.5, 0, Hq, Hkv, D, softcap=50.0)
+                actx.arena.release(m)
+            name = f"attention, bent scores, values of {n * D}, {kind}"
+            timed(name, attend, flops=2 * pairs * Hq * (D + n * D) if prompts else None,
+                  nbytes=None if prompts else R * 2048 * Hkv * (1 + n) * D * 2, like=None if n == 1 else f"attention, bent scores, values of {D}, {kind}")
+            out[name]["kernel"] = ops.last_attention_kernel
+    ops.check_device_status()
+    return {"rows": T, "width": W, "kernels": out}
 
 
 def pufivik_kernels_alone(torch, ops, peaks) -> dict:
@@ -871,7 +1024,8 @@ def compare_designs(args) -> int:
     bfloat16), and the device time of every class of operation in one eager step of each (CUDA events around every
     call, the calls of a class added up).  ``--compare besavik``: a Besavik model beside both.  ``--compare merudra``: a
     Merudra model beside a Besavik and a Qwen3 model.  ``--compare pufivik``: a Pufivik model beside a Merudra and a Qwen3
-    model.  ``--compare zugunex``: a Zugunex model beside a Besavik and a Qwen3 model.  Prints one JSON line."""
+    model.  ``--compare zugunex``: a Zugunex model beside a Besavik and a Qwen3 model.  ``--compare funudra``: a Funudra model
+    beside a Ganidra and a Qwen3 model.  Prints one JSON line."""
     import torch
     from qwen_engine_b200 import ops
     from qwen_engine_b200.config import preset_config_dict
@@ -985,23 +1139,27 @@ def compare_designs(args) -> int:
             out[name]["merudra"] = measure(config_from_dict(merudra_config_of(sz)), "merudra")
         if args.compare == "zugunex":
             out[name]["zugunex"] = measure(config_from_dict(zugunex_config_of(sz)), "zugunex")
+        if args.compare == "funudra":
+            out[name]["funudra"] = measure(config_from_dict(funudra_config_of(sz)), "funudra")
         if args.compare in ("besavik", "merudra", "zugunex"):
             out[name]["besavik"] = measure(config_from_dict(besavik_config_of(sz)), "besavik")
         if args.compare not in ("merudra", "pufivik", "zugunex"):
             out[name]["ganidra"] = measure(config_from_dict(ganidra_config_of(sz)), "ganidra")
         out[name]["qwen3"] = measure(config_from_dict(qraw), "qwen3")
-        designs = [d for d in ("zugunex", "pufivik", "merudra", "besavik", "ganidra", "qwen3") if d in out[name]]
+        designs = [d for d in ("funudra", "zugunex", "pufivik", "merudra", "besavik", "ganidra", "qwen3") if d in out[name]]
         for other in designs[1:]:
             g, q = out[name][designs[0]], out[name][other]
             out[name][f"{designs[0]}_over_{other}"] = {"prefill": round(g["prefill"]["tokens_per_s"] / q["prefill"]["tokens_per_s"], 3),
                                                       "decode": round(g["decode"]["tokens_per_s"] / q["decode"]["tokens_per_s"], 3)}
     alone = None
-    alone_of = {"merudra": merudra_kernels_alone, "pufivik": pufivik_kernels_alone, "zugunex": zugunex_kernels_alone}
+    alone_of = {"merudra": merudra_kernels_alone, "pufivik": pufivik_kernels_alone, "zugunex": zugunex_kernels_alone,
+                "funudra": funudra_kernels_alone}
     if not args.compare_size and args.compare in alone_of:
         alone = alone_of[args.compare](torch, ops, peaks)
     clocks.stop()
     title = {"besavik": "Besavik beside Ganidra and Qwen3", "merudra": "Merudra beside Besavik and Qwen3",
-             "pufivik": "Pufivik beside Merudra and Qwen3", "zugunex": "Zugunex beside Besavik and Qwen3"}.get(args.compare, "Ganidra beside Qwen3")
+             "pufivik": "Pufivik beside Merudra and Qwen3", "zugunex": "Zugunex beside Besavik and Qwen3",
+             "funudra": "Funudra beside Ganidra and Qwen3"}.get(args.compare, "Ganidra beside Qwen3")
     print(json.dumps({"metric": f"prefill and decode tok/s, {title} at equal sizes", "impl": "ours", "n_gpus": 1,
                       "dtype": "bf16", "data": "synthetic: uniform random token ids, random weights N(0, 0.02) seed 2",
                       "steps": args.steps, "warmup": args.warmup, "peaks": peaks_src, "sizes": out,
@@ -1030,9 +1188,9 @@ def main() -> int:
     ap.add_argument("--no-kernels", action="store_true", help="skip the per-kernel-class timings")
     ap.add_argument("--profile", choices=["decode", "prefill"], default=None,
                     help="bracket that timed region with cudaProfilerStart/Stop (for ncu --profile-from-start off)")
-    ap.add_argument("--compare", choices=["ganidra", "besavik", "merudra", "pufivik", "zugunex"], default=None,
+    ap.add_argument("--compare", choices=["ganidra", "besavik", "merudra", "pufivik", "zugunex", "funudra"], default=None,
                     help="instead of the default workload: prefill and decode of a Ganidra model beside a Qwen3 model of equal "
-                         "sizes (besavik: a Besavik model beside both; merudra: a Merudra model beside a Besavik and a Qwen3 model; pufivik: a Pufivik model beside a Merudra and a Qwen3 model; zugunex: a Zugunex model beside a Besavik and a Qwen3 model), with the device time of every class of operation "
+                         "sizes (besavik: a Besavik model beside both; merudra: a Merudra model beside a Besavik and a Qwen3 model; pufivik: a Pufivik model beside a Merudra and a Qwen3 model; zugunex: a Zugunex model beside a Besavik and a Qwen3 model; funudra: a Funudra model beside a Ganidra and a Qwen3 model), with the device time of every class of operation "
                          "(one JSON line)")
     ap.add_argument("--compare-size", choices=sorted(COMPARE_SIZES), default=None, help="with --compare: one size only")
     args = ap.parse_args()

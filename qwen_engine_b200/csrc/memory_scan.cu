@@ -14,10 +14,10 @@
 //
 // The scan: one CTA per (request, head, tile of value channels).  A value channel's column of S evolves on its own; a
 // thread owns J columns x DC consecutive key channels in registers, so that a staged q and k serve J columns; the L
-// threads of a column group are neighbours in one warp.  Every multiply-add works on a pair of channels.  Four producer
-// warps stage the next chunk of tokens in shared memory as float32; the first of them also forms the chunk's a and b (for
-// form 1 it carries m).  Four tokens a turn: their J sums each are exchanged together (a lane ends up with its share).
-// The order of every sum depends on the sizes alone, so a token's output does not depend on how its request was cut.
+// threads of a column group are neighbours in one warp.  Every multiply-add works on a pair of channels.  Chunks of tokens
+// come through a ring in shared memory (16-byte asynchronous copies, as they are stored); one more warp forms the next
+// chunk's a and b (for form 1 it carries m).  A few tokens a turn: their J sums each are exchanged together (a lane ends up
+// with its share).  The order of every sum depends on the sizes alone, so a token's output does not depend on how its request was cut.
 //
 // Steps of single tokens take a kernel of their own: nothing is staged, a thread's part of the state is on its way before
 // the kernel waits for the one before it.
@@ -27,9 +27,10 @@
 #include "common.cuh"
 #include <math.h>
 
-#define MS_COMPUTE 128
-#define MS_PRODUCERS 128
+#define MS_STAGES 3                // chunks of tokens in shared memory
 #define MS_SMEM_MAX (110 * 1024)
+__host__ __device__ constexpr int ms_threads_max(int J) { return J == 2 ? 256 : 128; }   // threads that hold state, at most
+__host__ __device__ constexpr int ms_turn(int J) { return J == 4 ? 4 : 8; }      // tokens whose sums are exchanged together
 
 struct MsArgs {
   const void* q; const void* k; const void* v; long ldq, ldk, ldv;
@@ -76,25 +77,18 @@ __device__ __forceinline__ float ms_softplus(float z) { return fmaxf(z, 0.f) + l
 
 // one token on a thread's J columns of DC channels: the state moves on, acc = q . s
 template <int DC, int J>
-__device__ __forceinline__ void ms_token(float2 (&s)[J][DC / 2], const float* qr, const float* kr, const float (&u)[J], float a,
-                                         float (&acc)[J]) {
+__device__ __forceinline__ void ms_token(float2 (&s)[J][DC / 2], const float2 (&q)[DC / 2], const float2 (&k)[DC / 2], const float (&u)[J],
+                                         float a, float (&acc)[J]) {
   float2 sum[J];
 #pragma unroll
   for (int j = 0; j < J; ++j) sum[j] = make_float2(0.f, 0.f);
   const float2 a2 = make_float2(a, a);
 #pragma unroll
-  for (int i = 0; i < DC; i += 4) {
-    const float4 q4 = *reinterpret_cast<const float4*>(qr + i);
-    const float4 k4 = *reinterpret_cast<const float4*>(kr + i);
+  for (int i = 0; i < DC / 2; ++i) {
 #pragma unroll
     for (int j = 0; j < J; ++j) {
-      const float2 u2 = make_float2(u[j], u[j]);
-      float2& s0 = s[j][i / 2];
-      float2& s1 = s[j][i / 2 + 1];
-      s0 = ms_fma2(a2, s0, ms_mul2(make_float2(k4.x, k4.y), u2));
-      s1 = ms_fma2(a2, s1, ms_mul2(make_float2(k4.z, k4.w), u2));
-      sum[j] = ms_fma2(make_float2(q4.x, q4.y), s0, sum[j]);
-      sum[j] = ms_fma2(make_float2(q4.z, q4.w), s1, sum[j]);
+      s[j][i] = ms_fma2(a2, s[j][i], ms_mul2(k[i], make_float2(u[j], u[j])));
+      sum[j] = ms_fma2(q[i], s[j][i], sum[j]);
     }
   }
 #pragma unroll
@@ -151,22 +145,59 @@ __device__ __forceinline__ void ms_store_state(const float2 (&s)[J][DC / 2], flo
   }
 }
 
-// index of key channel c in a staged row: blocks of DC channels with 4 floats between them (banks)
-template <int DC> __device__ __forceinline__ int ms_pad(int c) { return c + (c / DC) * 4; }
+// DC consecutive elements of the compute type in shared memory as pairs of floats
+template <int DC> __device__ __forceinline__ void ms_pairs(const __nv_bfloat16* p, float2 (&f)[DC / 2]) {
+#pragma unroll
+  for (int i = 0; i < DC / 8; ++i) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p + 8 * i);
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int x = 0; x < 4; ++x) f[4 * i + x] = make_float2(__uint_as_float(w[x] << 16), __uint_as_float(w[x] & 0xffff0000u));
+  }
+}
+template <int DC> __device__ __forceinline__ void ms_pairs(const float* p, float2 (&f)[DC / 2]) {
+#pragma unroll
+  for (int i = 0; i < DC / 4; ++i) {
+    const float4 r = *reinterpret_cast<const float4*>(p + 4 * i);
+    f[2 * i] = make_float2(r.x, r.y); f[2 * i + 1] = make_float2(r.z, r.w);
+  }
+}
+template <int J> __device__ __forceinline__ void ms_values(const __nv_bfloat16* p, float (&v)[J]) {
+  if constexpr (J == 4) {
+    const uint2 r = *reinterpret_cast<const uint2*>(p);
+    v[0] = __uint_as_float(r.x << 16); v[1] = __uint_as_float(r.x & 0xffff0000u);
+    v[2] = __uint_as_float(r.y << 16); v[3] = __uint_as_float(r.y & 0xffff0000u);
+  } else if constexpr (J == 2) {
+    const uint32_t r = *reinterpret_cast<const uint32_t*>(p);
+    v[0] = __uint_as_float(r << 16); v[1] = __uint_as_float(r & 0xffff0000u);
+  } else v[0] = __bfloat162float(p[0]);
+}
+template <int J> __device__ __forceinline__ void ms_values(const float* p, float (&v)[J]) {
+  if constexpr (J == 4) { const float4 r = *reinterpret_cast<const float4*>(p); v[0] = r.x; v[1] = r.y; v[2] = r.z; v[3] = r.w; }
+  else if constexpr (J == 2) { const float2 r = *reinterpret_cast<const float2*>(p); v[0] = r.x; v[1] = r.y; }
+  else v[0] = p[0];
+}
+// 16 bytes to shared memory; not valid: nothing is read and zeros are written
+__device__ __forceinline__ void ms_cp_async16(void* smem, const void* gmem, bool valid) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" :: "r"((uint32_t)__cvta_generic_to_shared(smem)), "l"(gmem), "r"(valid ? 16 : 0));
+}
 
 template <typename T, int DC, int J, int L>
-__global__ void __launch_bounds__(MS_COMPUTE + MS_PRODUCERS)
+__global__ void __launch_bounds__(ms_threads_max(J) + 32, 1)
 memory_scan_kernel(MsArgs A) {
-  extern __shared__ __align__(16) float smem[];
+  extern __shared__ __align__(16) unsigned char smem_raw[];
   const int req = blockIdx.x, head = blockIdx.y, VT = A.VT, j0 = blockIdx.z * VT;
-  const int dk = A.dk, dv = A.dv, dvx = A.dvx, H = A.H;
-  constexpr int row_w = L * (DC + 4);
-  const int VTp = (VT + 3) & ~3;
-  const int tok_w = 2 * row_w + VTp + 4;                // q, k, v of the tile, (a, b, exp(-m))
-  auto buf = [&](int ch) { return smem + (size_t)(ch & 1) * A.chunk * tok_w; };
-  const int n_compute = blockDim.x - MS_PRODUCERS;
-  const int tid = threadIdx.x;
-  const bool producer = tid >= n_compute;
+  const int dk = A.dk, dv = A.dv, dvx = A.dvx, H = A.H, chunk = A.chunk;
+  constexpr int QW = L * DC;                            // elements of a staged row of q or k
+  constexpr int VEC = 16 / (int)sizeof(T);
+  constexpr int TURN = ms_turn(J);
+  const int VTp = (VT + VEC - 1) / VEC * VEC;
+  const int stage_elems = chunk * (2 * QW + VTp);       // q rows, k rows, v rows
+  T* const stages = reinterpret_cast<T*>(smem_raw);
+  float4* const scalars = reinterpret_cast<float4*>(stages + (size_t)MS_STAGES * stage_elems);       // [2][chunk]: a, b, exp(-m)
+  const int n_compute = blockDim.x - 32;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const bool scalar_warp = tid >= n_compute;
   const int l = tid % L, cg = tid / L;
   const int jc = j0 + cg * J;                           // the thread's first column
   const int j_end = min(dvx, j0 + VT);
@@ -175,166 +206,150 @@ memory_scan_kernel(MsArgs A) {
   const int n = A.cu_q[req + 1] - row0;
   const int ctx = A.ctx_lens[req], slot = A.slot_ids[req];
   if (n <= 0) { pdl_wait(); return; }
-  const int n_chunks = (n + A.chunk - 1) / A.chunk;
-  const int chunk = A.chunk;
+  const int n_chunks = (n + chunk - 1) / chunk;
   float* st = A.state + ((size_t)slot * H + head) * dvx * dk;
   float* ms = A.mstate ? A.mstate + ((size_t)slot * H + head) * dvx : nullptr;
 
-  if (producer) {
-    const int ptid = tid - n_compute, plane_ = tid & 31;
-    const int grp = head / (H / A.G);
-    const T* q = (const T*)A.q + (size_t)grp * dk;
-    const T* k = (const T*)A.k + (size_t)grp * dk;
-    const T* v = (const T*)A.v + (size_t)head * dv;
+  if (scalar_warp) {
+    // ---- a and b of a chunk's tokens, a token a lane; form 1 carries m through them one after the other ----------
     const float bias0 = A.b0 ? A.b0[head] : 0.f, bias1 = A.b1 ? A.b1[head] : 0.f;
     const float rate = A.log_rate ? expf(A.log_rate[head]) : 0.f;
     float m = (A.form == 1 && ctx > 0) ? ms[j0] : 0.f;
-    // what no copy writes: key channels beyond the head, in both buffers
-    if (L * DC > dk)
-      for (int e = ptid; e < 2 * chunk * (L * DC - dk); e += MS_PRODUCERS) {
-        const int t = e / (L * DC - dk), c = dk + e - t * (L * DC - dk);
-        float* dst = smem + (size_t)t * tok_w + ms_pad<DC>(c);
-        dst[0] = 0.f; dst[row_w] = 0.f;
-      }
     pdl_wait();
-    constexpr int VEC = 16 / (int)sizeof(T);
-    auto stage = [&](int ch) {
-      float* b = buf(ch);
-      const int t_first = ch * chunk, rows = min(chunk, n - t_first), rows4 = min((rows + 3) & ~3, chunk);
-      // a and b of the chunk's tokens: one warp, a token a lane (32 at most a turn)
-      if (ptid < 32) {
-        for (int tb = 0; tb < rows4; tb += 32) {
-          const int t = tb + plane_;
-          float a = 1.f, bb = 0.f, fl = 0.f;
-          const size_t row = (size_t)(row0 + t_first + t);
-          if (A.form == 0) {
-            if (t < rows) {
-              const float dt = ms_softplus(ms_gate_in<T>(A.g0, A.ldg0, A.gates_f32, row, head) + bias0);
-              a = expf(-rate * dt); bb = dt;
-            }
-          } else {
-            float gi = 0.f, gf = 0.f;
-            if (t < rows) {
-              gi = ms_log_in(ms_gate_in<T>(A.g0, A.ldg0, A.gates_f32, row, head) + bias0, A.cap);
-              gf = ms_log_keep(ms_gate_in<T>(A.g1, A.ldg1, A.gates_f32, row, head) + bias1, A.cap);
-            }
-            float kept = 0.f, mine = 0.f;
-            const int n_here = min(32, rows - tb);
-            for (int x = 0; x < n_here; ++x) {
-              const float fx = __shfl_sync(0xffffffffu, gf, x), ix = __shfl_sync(0xffffffffu, gi, x);
-              const float kx = fx + m;
-              m = fmaxf(kx, ix);
-              if (x == plane_) { kept = kx; mine = m; }
-            }
-            if (t < rows) { a = expf(kept - mine); bb = expf(gi - mine); fl = expf(-mine); }
+    auto form_chunk = [&](int ch) {
+      const int t_first = ch * chunk, rows = min(chunk, n - t_first);
+      for (int tb = 0; tb < chunk; tb += 32) {
+        const int t = tb + lane;
+        float a = 1.f, bb = 0.f, fl = 0.f;              // (tokens behind the last: nothing decays, nothing comes in)
+        const size_t row = (size_t)(row0 + t_first + t);
+        if (A.form == 0) {
+          if (t < rows) {
+            bb = ms_softplus(ms_gate_in<T>(A.g0, A.ldg0, A.gates_f32, row, head) + bias0);
+            a = expf(-rate * bb);
           }
-          if (t < rows4) *reinterpret_cast<float4*>(b + (size_t)t * tok_w + 2 * row_w + VTp) = make_float4(a, bb, fl, 0.f);
+        } else {
+          float gi = 0.f, gf = 0.f;
+          if (t < rows) {
+            gi = ms_log_in(ms_gate_in<T>(A.g0, A.ldg0, A.gates_f32, row, head) + bias0, A.cap);
+            gf = ms_log_keep(ms_gate_in<T>(A.g1, A.ldg1, A.gates_f32, row, head) + bias1, A.cap);
+          }
+          float kept = 0.f, mine = 0.f;
+          const int n_here = min(32, rows - tb);
+          for (int x = 0; x < n_here; ++x) {
+            const float fx = __shfl_sync(0xffffffffu, gf, x), ix = __shfl_sync(0xffffffffu, gi, x);
+            const float kx = fx + m;
+            m = fmaxf(kx, ix);
+            if (x == lane) { kept = kx; mine = m; }
+          }
+          if (t < rows) { a = expf(kept - mine); bb = expf(gi - mine); fl = expf(-mine); }
         }
-      }
-      if (A.vec) {
-        // pieces of 16 bytes: q, k of the group, v of the tile; several loads on their way before the first is stored
-        const int pk = dk / VEC, pv = VT / VEC, per = 2 * pk + pv;
-        const int total = rows * per;
-        constexpr int NI = 4;
-        for (int e0 = ptid; e0 < total; e0 += NI * MS_PRODUCERS) {
-          uint4 r[NI];
-          int dst[NI], kind[NI];
-#pragma unroll
-          for (int i = 0; i < NI; ++i) {
-            const int e = e0 + i * MS_PRODUCERS;
-            kind[i] = -1;
-            if (e >= total) continue;
-            const int t = e / per;
-            int x = e - t * per;
-            const size_t row = (size_t)(row0 + t_first + t);
-            const T* src;
-            if (x < pk) { kind[i] = 0; src = q + row * A.ldq + x * VEC; dst[i] = t * tok_w + ms_pad<DC>(x * VEC); }
-            else if ((x -= pk) < pk) { kind[i] = 1; src = k + row * A.ldk + x * VEC; dst[i] = t * tok_w + row_w + ms_pad<DC>(x * VEC); }
-            else {
-              x -= pk;
-              kind[i] = 2; dst[i] = t * tok_w + 2 * row_w + x * VEC;
-              src = v + row * A.ldv + j0 + x * VEC;
-              if (j0 + x * VEC >= dv) { kind[i] = j0 + x * VEC == dv ? 3 : 4; continue; }     // the normaliser's column, or beyond
-            }
-            r[i] = __ldg(reinterpret_cast<const uint4*>(src));
-          }
-#pragma unroll
-          for (int i = 0; i < NI; ++i) {
-            if (kind[i] < 0) continue;
-            float f[VEC];
-            if (kind[i] >= 3) {
-#pragma unroll
-              for (int x = 0; x < VEC; ++x) f[x] = (kind[i] == 3 && x == 0) ? 1.f : 0.f;
-            } else if constexpr (sizeof(T) == 2) {
-              const __nv_bfloat162* h2 = reinterpret_cast<const __nv_bfloat162*>(&r[i]);
-#pragma unroll
-              for (int x = 0; x < 4; ++x) { const float2 y = __bfloat1622float2(h2[x]); f[2 * x] = y.x; f[2 * x + 1] = y.y; }
-            } else {
-              f[0] = __uint_as_float(r[i].x); f[1] = __uint_as_float(r[i].y); f[2] = __uint_as_float(r[i].z); f[3] = __uint_as_float(r[i].w);
-            }
-            if (kind[i] == 0) {
-#pragma unroll
-              for (int x = 0; x < VEC; ++x) f[x] *= A.q_scale;
-            }
-            // (a piece lies within one block of DC channels: DC is a multiple of VEC)
-            *reinterpret_cast<float4*>(b + dst[i]) = make_float4(f[0], f[1], f[2], f[3]);
-            if constexpr (VEC == 8) *reinterpret_cast<float4*>(b + dst[i] + 4) = make_float4(f[4], f[5], f[6], f[7]);
-          }
-        }
-      } else {
-        const int per = 2 * dk + VT;
-        for (int e = ptid; e < rows * per; e += MS_PRODUCERS) {
-          const int t = e / per;
-          int x = e - t * per;
-          const size_t row = (size_t)(row0 + t_first + t);
-          float* dst = b + (size_t)t * tok_w;
-          if (x < dk) dst[ms_pad<DC>(x)] = to_f32(q[row * A.ldq + x]) * A.q_scale;
-          else if ((x -= dk) < dk) dst[row_w + ms_pad<DC>(x)] = to_f32(k[row * A.ldk + x]);
-          else {
-            x -= dk;
-            dst[2 * row_w + x] = j0 + x < dv ? to_f32(v[row * A.ldv + j0 + x]) : (j0 + x == dv ? 1.f : 0.f);
-          }
-        }
-      }
-      // tokens that fill the last turn of four: nothing in, nothing decays (their outputs are not stored)
-      for (int e = ptid; e < (rows4 - rows) * (2 * row_w + VTp); e += MS_PRODUCERS) {
-        const int t = e / (2 * row_w + VTp), x = e - t * (2 * row_w + VTp);
-        b[(size_t)(rows + t) * tok_w + x] = 0.f;
+        if (t < chunk) scalars[(ch & 1) * chunk + t] = make_float4(a, bb, fl, 0.f);
       }
     };
-    stage(0);
-    __syncthreads();
+    form_chunk(0);
     for (int ch = 0; ch < n_chunks; ++ch) {
-      if (ch + 1 < n_chunks) stage(ch + 1);
       __syncthreads();
+      if (ch + 1 < n_chunks) form_chunk(ch + 1);
     }
-    if (A.form == 1 && A.write_state && ptid < 32)
-      for (int j = j0 + plane_; j < j_end; j += 32) ms[j] = m;
+    if (A.form == 1 && A.write_state)
+      for (int j = j0 + lane; j < j_end; j += 32) ms[j] = m;
     return;
   }
 
   // ---- the columns ----------------------------------------------------------------------------------------
+  const int grp = head / (H / A.G);
+  const T* q = (const T*)A.q + (size_t)grp * dk;
+  const T* k = (const T*)A.k + (size_t)grp * dk;
+  const T* v = (const T*)A.v + (size_t)head * dv;
+  // what no copy writes, in every stage: key channels beyond the head (zero), the normaliser's value (one) and what lies
+  // behind it (zero)
+  {
+    const int extra_k = QW - dk, v_first = min(VTp, max(0, dv - j0)), extra_v = VTp - v_first, per = 2 * extra_k + extra_v;
+    if (per > 0)
+      for (int e = tid; e < MS_STAGES * chunk * per; e += n_compute) {
+        const int t = e / per, s = t / chunk, r = t - s * chunk;
+        int x = e - t * per;
+        T* base = stages + (size_t)s * stage_elems;
+        if (x < extra_k) base[(size_t)r * QW + dk + x] = from_f32<T>(0.f);
+        else if ((x -= extra_k) < extra_k) base[(size_t)(chunk + r) * QW + dk + x] = from_f32<T>(0.f);
+        else {
+          x += v_first - extra_k;
+          base[(size_t)2 * chunk * QW + (size_t)r * VTp + x] = from_f32<T>(j0 + x == dv ? 1.f : 0.f);
+        }
+      }
+  }
   float2 s[J][DC / 2];
   ms_load_state<DC, J>(s, st, dk, l, jc, j_end, ctx > 0);
-  float skip = A.skip ? A.skip[head] : 0.f;
+  const float skip = A.skip ? A.skip[head] : 0.f, q_scale = A.q_scale;
   pdl_wait();
-  __syncthreads();
+  // a chunk's rows of q, k (the group's) and v (the tile's): pieces of 16 bytes, a thread keeps to one place of the row
+  const int pk = dk / VEC, pv = min(VT, max(0, dv - j0)) / VEC, per = 2 * pk + pv;
+  const int at_once = max(1, n_compute / max(1, per)), my_row = per <= n_compute ? tid / max(1, per) : 0;
+  auto issue = [&](int ch) {
+    if (ch < n_chunks) {
+      T* base = stages + (size_t)(ch % MS_STAGES) * stage_elems;
+      const int t_first = ch * chunk, rows = min(chunk, n - t_first);
+      if (A.vec) {
+        if (my_row < at_once)
+          for (int x = per <= n_compute ? tid - my_row * per : tid; x < per; x += n_compute) {
+            const T* src; T* dst; long ld; int pitch;
+            if (x < pk) { src = q + x * VEC; ld = A.ldq; dst = base + x * VEC; pitch = QW; }
+            else if (x < 2 * pk) { src = k + (x - pk) * VEC; ld = A.ldk; dst = base + (size_t)chunk * QW + (x - pk) * VEC; pitch = QW; }
+            else { src = v + j0 + (x - 2 * pk) * VEC; ld = A.ldv; dst = base + (size_t)2 * chunk * QW + (x - 2 * pk) * VEC; pitch = VTp; }
+            src += (size_t)(row0 + t_first + my_row) * ld;
+            dst += my_row * pitch;
+            const long src_step = (long)at_once * ld;
+            const int dst_step = at_once * pitch;
+            for (int t = my_row; t < chunk; t += at_once, dst += dst_step) {
+              ms_cp_async16(dst, t < rows ? src : q, t < rows);
+              src += src_step;
+            }
+          }
+      } else {
+        const int ev = min(VT, max(0, dv - j0)), pe = 2 * dk + ev;
+        for (int e = tid; e < chunk * pe; e += n_compute) {
+          const int t = e / pe;
+          int x = e - t * pe;
+          const size_t row = (size_t)(row0 + t_first + t);
+          const bool in = t < rows;
+          if (x < dk) base[(size_t)t * QW + x] = in ? q[row * A.ldq + x] : from_f32<T>(0.f);
+          else if ((x -= dk) < dk) base[(size_t)(chunk + t) * QW + x] = in ? k[row * A.ldk + x] : from_f32<T>(0.f);
+          else {
+            x -= dk;
+            base[(size_t)2 * chunk * QW + (size_t)t * VTp + x] = in ? v[row * A.ldv + j0 + x] : from_f32<T>(0.f);
+          }
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;\n" ::: "memory");
+  };
+  for (int ch = 0; ch < MS_STAGES - 1; ++ch) issue(ch);
   const size_t o_ld = (size_t)H * dv;
   for (int ch = 0; ch < n_chunks; ++ch) {
+    asm volatile("cp.async.wait_group %0;\n" :: "n"(MS_STAGES - 2) : "memory");
+    __syncthreads();                                    // the chunk and its scalars are there; nobody reads the stage that is filled next
+    issue(ch + MS_STAGES - 1);
     const int rows = min(chunk, n - ch * chunk);
-    const float* r = buf(ch);
+    const T* base = stages + (size_t)(ch % MS_STAGES) * stage_elems;
+    const T* qp = base + l * DC;
+    const T* kp = base + (size_t)chunk * QW + l * DC;
+    const T* vp = base + (size_t)2 * chunk * QW + cg * J;
+    const float4* sc = scalars + (ch & 1) * chunk;
     const size_t row = (size_t)(row0 + ch * chunk);
-    for (int t0 = 0; t0 < rows; t0 += 4, r += 4 * tok_w) {
-      constexpr int NV = 4 * J;
+    for (int t0 = 0; t0 < rows; t0 += TURN) {
+      constexpr int NV = TURN * J;
       float val[NV];                                    // [token][column]
 #pragma unroll
-      for (int t = 0; t < 4; ++t) {
-        const float* rt = r + t * tok_w;
-        const float2 ab = *reinterpret_cast<const float2*>(rt + 2 * row_w + VTp);
-        float u[J], acc[J];
+      for (int t = 0; t < TURN; ++t) {
+        const float2 ab = *reinterpret_cast<const float2*>(sc + t0 + t);
+        float2 qf[DC / 2], kf[DC / 2];
+        float vv[J], u[J], acc[J];
+        ms_pairs<DC>(qp + (size_t)(t0 + t) * QW, qf);
+        ms_pairs<DC>(kp + (size_t)(t0 + t) * QW, kf);
+        ms_values<J>(vp + (size_t)(t0 + t) * VTp, vv);
 #pragma unroll
-        for (int j = 0; j < J; ++j) u[j] = ab.y * rt[2 * row_w + cg * J + j];
-        ms_token<DC, J>(s, rt + l * (DC + 4), rt + row_w + l * (DC + 4), u, ab.x, acc);
+        for (int j = 0; j < J; ++j) u[j] = ab.y * vv[j];
+        ms_token<DC, J>(s, qf, kf, u, ab.x, acc);
 #pragma unroll
         for (int j = 0; j < J; ++j) val[t * J + j] = acc[j];
       }
@@ -363,20 +378,19 @@ memory_scan_kernel(MsArgs A) {
           if (i >= held) continue;
           const int x = mine + i, t = x / J, j = x - t * J, col = jc + j;
           if (t0 + t >= rows || col >= j_end) continue;
-          const float* rt = r + t * tok_w;
-          if (col < dv) A.out[(row + t0 + t) * o_ld + (size_t)head * dv + col] = fmaf(skip, rt[2 * row_w + cg * J + j], val[i]);
-          else A.den[(row + t0 + t) * H + head] = fmaxf(fabsf(val[i]), rt[2 * row_w + VTp + 2]) + A.den_eps;
+          const float y = val[i] * q_scale;
+          if (col < dv) A.out[(row + t0 + t) * o_ld + (size_t)head * dv + col] = A.skip ? fmaf(skip, to_f32(vp[(size_t)(t0 + t) * VTp + j]), y) : y;
+          else A.den[(row + t0 + t) * H + head] = fmaxf(fabsf(y), sc[t0 + t].z) + A.den_eps;
         }
       }
     }
-    __syncthreads();
   }
   if (A.write_state) ms_store_state<DC, J>(s, st, dk, l, jc, j_end);
 }
 
 // A step of single tokens: one token a request.
 template <typename T, int DC, int J, int L>
-__global__ void __launch_bounds__(MS_COMPUTE)
+__global__ void __launch_bounds__(ms_threads_max(J))
 memory_step_kernel(MsArgs A) {
   const int req = blockIdx.x, head = blockIdx.y, j0 = blockIdx.z * A.VT;
   const int dk = A.dk, dv = A.dv, dvx = A.dvx, H = A.H;
@@ -400,12 +414,12 @@ memory_step_kernel(MsArgs A) {
   const T* q = (const T*)A.q + row * A.ldq + (size_t)grp * dk;
   const T* k = (const T*)A.k + row * A.ldk + (size_t)grp * dk;
   const T* v = (const T*)A.v + row * A.ldv + (size_t)head * dv;
-  float qf[DC], kf[DC];
+  float2 qf[DC / 2], kf[DC / 2];
 #pragma unroll
-  for (int i = 0; i < DC; ++i) {
-    const int c = l * DC + i;
-    qf[i] = c < dk ? to_f32(q[c]) * A.q_scale : 0.f;
-    kf[i] = c < dk ? to_f32(k[c]) : 0.f;
+  for (int i = 0; i < DC / 2; ++i) {
+    const int c = l * DC + 2 * i;
+    qf[i] = make_float2(c < dk ? to_f32(q[c]) : 0.f, c + 1 < dk ? to_f32(q[c + 1]) : 0.f);
+    kf[i] = make_float2(c < dk ? to_f32(k[c]) : 0.f, c + 1 < dk ? to_f32(k[c + 1]) : 0.f);
   }
   float vf[J];
 #pragma unroll
@@ -433,8 +447,9 @@ memory_step_kernel(MsArgs A) {
     for (int j = 0; j < J; ++j) {
       const int col = jc + j;
       if (col >= j_end) continue;
-      if (col < dv) A.out[row * ((size_t)H * dv) + (size_t)head * dv + col] = fmaf(skip, vf[j], acc[j]);
-      else A.den[row * H + head] = fmaxf(fabsf(acc[j]), fl) + A.den_eps;
+      const float y = acc[j] * A.q_scale;
+      if (col < dv) A.out[row * ((size_t)H * dv) + (size_t)head * dv + col] = A.skip ? fmaf(skip, vf[j], y) : y;
+      else A.den[row * H + head] = fmaxf(fabsf(y), fl) + A.den_eps;
     }
   }
   if (A.write_state) {
@@ -444,9 +459,9 @@ memory_step_kernel(MsArgs A) {
   }
 }
 
-// The columns of a CTA: as many as MS_COMPUTE threads hold, fewer where the grid would leave SMs idle.
+// The columns of a CTA: as many as its threads hold at most, fewer where the grid would leave SMs idle.
 static int ms_threads(long units, int dvx, int L, int J) {
-  int threads = MS_COMPUTE;
+  int threads = ms_threads_max(J);
   auto tiles = [&](int th) { const int vt = th / L * J; return (long)((dvx + vt - 1) / vt); };
   while (threads > 32 && threads / 2 / L * J >= 8 && (units * tiles(threads) < 148 || threads / 2 / L * J >= dvx)) threads /= 2;
   return threads;
@@ -463,13 +478,13 @@ static int ms_launch(MsArgs A, int R, int max_q_len, cudaStream_t stream) {
     QE_CHECK_LAUNCH("memory_scan");
     return 0;
   }
-  const int tok_w = 2 * L * (DC + 4) + ((A.VT + 3) & ~3) + 4;
+  const int VEC = 16 / (int)sizeof(T);
+  const size_t token = (size_t)MS_STAGES * (2 * L * DC + (A.VT + VEC - 1) / VEC * VEC) * sizeof(T) + 2 * sizeof(float4);
   int chunk = 32;
-  while (chunk > 4 && ((size_t)2 * chunk * tok_w * 4 > MS_SMEM_MAX || chunk / 2 >= max_q_len)) chunk >>= 1;
-  const size_t smem = (size_t)2 * chunk * tok_w * 4;
+  while (chunk > ms_turn(J) && (chunk * token > MS_SMEM_MAX || chunk / 2 >= max_q_len)) chunk >>= 1;
+  const size_t smem = chunk * token;
   if (smem > MS_SMEM_MAX) QE_REFUSE("memory_scan: key size %d needs %zu bytes of shared memory", A.dk, smem);
   A.chunk = chunk;
-  const int VEC = 16 / (int)sizeof(T);
   A.vec = A.dk % VEC == 0 && A.dv % VEC == 0 && A.VT % VEC == 0 && A.ldq % VEC == 0 && A.ldk % VEC == 0 && A.ldv % VEC == 0 &&
           (((uintptr_t)A.q | (uintptr_t)A.k | (uintptr_t)A.v) & 15) == 0;
   static bool configured = false;
@@ -478,7 +493,7 @@ static int ms_launch(MsArgs A, int R, int max_q_len, cudaStream_t stream) {
     if (e != cudaSuccess) QE_REFUSE("memory_scan: shared memory: %s", cudaGetErrorString(e));
     configured = true;
   }
-  qe_launch(memory_scan_kernel<T, DC, J, L>, grid, dim3(threads + MS_PRODUCERS), smem, stream, A);
+  qe_launch(memory_scan_kernel<T, DC, J, L>, grid, dim3(threads + 32), smem, stream, A);
   QE_CHECK_LAUNCH("memory_scan");
   return 0;
 }
@@ -502,15 +517,21 @@ extern "C" int qe_memory_scan(const void* q, long ldq, const void* k, long ldk, 
   int L = 1;
   const int DC = dk <= 256 ? 8 : 32;
   while (L * DC < dk) L <<= 1;
+  // Prompt portions in bfloat16 that fill the SMs only once: two columns a thread and twice the warps (latencies overlap);
+  // otherwise four columns a thread (fewer conversions and loads for the same state).  The bits are the same.
+  const bool few = max_q_len > 1 && dtype == QE_DTYPE_BF16 && DC == 8 && (long)R * H * ((A.dvx + 31) / 32) < 256;
+#define MSL_L(TT, JJ) do { switch (L) { \
+      case 1: return ms_launch<TT, 8, JJ, 1>(A, R, max_q_len, stream); case 2: return ms_launch<TT, 8, JJ, 2>(A, R, max_q_len, stream); \
+      case 4: return ms_launch<TT, 8, JJ, 4>(A, R, max_q_len, stream); case 8: return ms_launch<TT, 8, JJ, 8>(A, R, max_q_len, stream); \
+      case 16: return ms_launch<TT, 8, JJ, 16>(A, R, max_q_len, stream); default: return ms_launch<TT, 8, JJ, 32>(A, R, max_q_len, stream); } } while (0)
 #define MSL(TT) do { \
-    if (DC == 8) switch (L) { \
-      case 1: return ms_launch<TT, 8, 4, 1>(A, R, max_q_len, stream); case 2: return ms_launch<TT, 8, 4, 2>(A, R, max_q_len, stream); \
-      case 4: return ms_launch<TT, 8, 4, 4>(A, R, max_q_len, stream); case 8: return ms_launch<TT, 8, 4, 8>(A, R, max_q_len, stream); \
-      case 16: return ms_launch<TT, 8, 4, 16>(A, R, max_q_len, stream); default: return ms_launch<TT, 8, 4, 32>(A, R, max_q_len, stream); } \
-    else switch (L) { case 16: return ms_launch<TT, 32, 1, 16>(A, R, max_q_len, stream); default: return ms_launch<TT, 32, 1, 32>(A, R, max_q_len, stream); } \
+    if (DC == 8) MSL_L(TT, 4); \
+    switch (L) { case 16: return ms_launch<TT, 32, 1, 16>(A, R, max_q_len, stream); default: return ms_launch<TT, 32, 1, 32>(A, R, max_q_len, stream); } \
   } while (0)
+  if (few) MSL_L(__nv_bfloat16, 2);
   if (dtype == QE_DTYPE_F32) MSL(float);
-  else if (dtype == QE_DTYPE_BF16) MSL(__nv_bfloat16);
+  if (dtype == QE_DTYPE_BF16) MSL(__nv_bfloat16);
 #undef MSL
+#undef MSL_L
   QE_REFUSE("memory_scan: unknown dtype %d", dtype);
 }
