@@ -142,7 +142,7 @@ conv_act_kernel(ConvArgs A, const float* __restrict__ out_bias, T* __restrict__ 
   const bool has_ctx = A.ctx_lens[req] > 0;
   col.open(A, c, A.slot_ids[req], row0, t0, has_ctx);
   const int t1 = min(n, t0 + CV_TOKENS);
-  constexpr int AHEAD = 4;                           // inputs on their way at a time
+  constexpr int AHEAD = VEC == 4 ? 8 : 4;                           // inputs on their way at a time
   for (int t = t0; t < t1; t += AHEAD) {
     float u[AHEAD][VEC];
 #pragma unroll
@@ -155,7 +155,7 @@ conv_act_kernel(ConvArgs A, const float* __restrict__ out_bias, T* __restrict__ 
 #pragma unroll
       for (int i = 0; i < VEC; ++i) {
         y[i] += ob[i];
-        if (silu) y[i] = y[i] / (1.f + expf(-y[i]));
+        if (silu) y[i] = act_for<T>(y[i], 3);           // (the hardware's exponential and quotient where the result is rounded to bfloat16)
       }
       CvVec<T, VEC>::st(out + (size_t)(row0 + t + a) * ldo + c, y);
     }

@@ -160,10 +160,11 @@ struct GroupGateArgs {
   const float* x; long ldx; const void* g; long ldg; const float* w; const float* den; void* out; long ldo;
   float eps, scale; int G, D, gate, gate_first, items;      // G groups of D channels; gate 0 none, 1 silu, 2 sigmoid
 };
-__device__ __forceinline__ float nr_gate(float g, int kind) {
-  if (kind == 1) return g / (1.f + expf(-g));
-  if (kind == 2) return 1.f / (1.f + expf(-g));
-  return 1.f;
+// (bfloat16 results: the hardware's exponential and quotient)
+template <typename T> __device__ __forceinline__ float nr_gate(float g, int kind) {
+  if (kind == 0) return 1.f;
+  const float num = kind == 1 ? g : 1.f;
+  return sizeof(T) == 4 ? num / (1.f + expf(-g)) : __fdividef(num, 1.f + __expf(-g));
 }
 
 // WPG warps a group (1: eight groups a CTA; else the CTA is one group's), NV pieces of four channels a thread
@@ -203,7 +204,7 @@ __global__ void __launch_bounds__(256) group_norm_gate_kernel(GroupGateArgs A) {
     if (d >= D) continue;
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
-      if (g) gv[i][u] = nr_gate(gv[i][u], A.gate);
+      if (g) gv[i][u] = nr_gate<T>(gv[i][u], A.gate);
       if (A.den) v[i][u] = v[i][u] / div;
       if (A.gate_first && g) v[i][u] *= gv[i][u];
       ss = fmaf(v[i][u], v[i][u], ss);
@@ -239,7 +240,7 @@ __global__ void __launch_bounds__(128) group_norm_gate_plain_kernel(GroupGateArg
   const float div = A.den ? A.den[item] : 1.f;
   auto value = [&](int d) {
     float v = A.den ? x[d] / div : x[d];
-    if (A.gate_first && g) v *= nr_gate(to_f32(g[d]), A.gate);
+    if (A.gate_first && g) v *= nr_gate<T>(to_f32(g[d]), A.gate);
     return v;
   };
   float ss = 0.f;
@@ -249,7 +250,7 @@ __global__ void __launch_bounds__(128) group_norm_gate_plain_kernel(GroupGateArg
   T* out = (T*)A.out + (size_t)t * A.ldo + (size_t)gr * D;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float r = value(d) * rstd * A.w[(size_t)gr * D + d];
-    if (g && !A.gate_first) r *= nr_gate(to_f32(g[d]), A.gate);
+    if (g && !A.gate_first) r *= nr_gate<T>(to_f32(g[d]), A.gate);
     out[d] = from_f32<T>(r * A.scale);
   }
 }
