@@ -23,6 +23,13 @@
 template <typename T, int N> struct CvVec;
 template <> struct CvVec<float, 1> { static __device__ __forceinline__ void ld(const float* p, float (&f)[1]) { f[0] = *p; }
                                      static __device__ __forceinline__ void st(float* p, const float (&f)[1]) { *p = f[0]; } };
+template <> struct CvVec<float, 2> {
+  static __device__ __forceinline__ void ld(const float* p, float (&f)[2]) { const float2 v = *reinterpret_cast<const float2*>(p); f[0] = v.x; f[1] = v.y; }
+  static __device__ __forceinline__ void st(float* p, const float (&f)[2]) { *reinterpret_cast<float2*>(p) = make_float2(f[0], f[1]); } };
+template <> struct CvVec<__nv_bfloat16, 2> {
+  static __device__ __forceinline__ void ld(const __nv_bfloat16* p, float (&f)[2]) {
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); f[0] = a.x; f[1] = a.y; }
+  static __device__ __forceinline__ void st(__nv_bfloat16* p, const float (&f)[2]) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[1]); } };
 template <> struct CvVec<float, 4> {
   static __device__ __forceinline__ void ld(const float* p, float (&f)[4]) {
     const float4 v = *reinterpret_cast<const float4*>(p); f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w; }
@@ -123,7 +130,7 @@ struct ConvColumn {
 
 // ---------------------------------------------------------------------------------------------------------
 template <typename T, int VEC, int MT>
-__global__ void __launch_bounds__(CV_THREADS)
+__global__ void __launch_bounds__(CV_THREADS, MT == 4 ? 8 : 1)
 conv_act_kernel(ConvArgs A, const float* __restrict__ out_bias, T* __restrict__ out, long ldo, int silu) {
   pdl_launch_dependents();
   const int c = (blockIdx.x * CV_THREADS + threadIdx.x) * VEC, req = blockIdx.y, t0 = blockIdx.z * CV_TOKENS;
@@ -142,7 +149,7 @@ conv_act_kernel(ConvArgs A, const float* __restrict__ out_bias, T* __restrict__ 
   const bool has_ctx = A.ctx_lens[req] > 0;
   col.open(A, c, A.slot_ids[req], row0, t0, has_ctx);
   const int t1 = min(n, t0 + CV_TOKENS);
-  constexpr int AHEAD = VEC == 4 ? 8 : 4;                           // inputs on their way at a time
+  constexpr int AHEAD = 2;                           // inputs on their way at a time (warps hide the latency: more of them beat more loads a thread)
   for (int t = t0; t < t1; t += AHEAD) {
     float u[AHEAD][VEC];
 #pragma unroll
@@ -174,7 +181,7 @@ struct ConvQkvArgs {
 // A thread owns two pieces of VEC channels of one head: the two sides of the pairs that turn together, or two pieces of
 // the channels that do not turn.
 template <typename T, int VEC, int MT>
-__global__ void __launch_bounds__(CV_THREADS)
+__global__ void __launch_bounds__(CV_THREADS, MT == 4 ? 8 : 1)
 conv_qkv_kernel(ConvArgs A, ConvQkvArgs Q) {
   pdl_launch_dependents();
   const int D = Q.D, per_head = D / 2 / VEC;
@@ -201,7 +208,7 @@ conv_qkv_kernel(ConvArgs A, ConvQkvArgs Q) {
   const int vh = head - Q.H - Q.Hkv;
   const int plane = is_v ? 1 + vh % Q.VP : 0, hkv = is_v ? vh / Q.VP : head - Q.H;
   const int t1 = min(n, t0 + CV_TOKENS);
-  constexpr int AHEAD = 4;
+  constexpr int AHEAD = 2;
   for (int t = t0; t < t1; t += AHEAD) {
     float ua[AHEAD][VEC], ub[AHEAD][VEC];
 #pragma unroll
@@ -283,13 +290,13 @@ extern "C" int qe_conv_qkv(const void* x, long ldx, const float* in_bias, const 
   if (dtype != QE_DTYPE_F32 && dtype != QE_DTYPE_BF16) QE_REFUSE("conv_qkv: unknown dtype %d", dtype);
   const size_t es = dtype == QE_DTYPE_F32 ? 4 : 2;
   ConvQkvArgs Q{positions, inv_freq, (const float2*)cos_sin, q, ldq, pages, slot_mapping, H, Hkv, value_planes, D, rot_dims, page_size};
-  const bool vec = conv_aligned(A, es) && D % 8 == 0 && rot_dims % 8 == 0 && ldq % 4 == 0 && ((uintptr_t)q % (4 * es)) == 0 &&
+  const bool vec = conv_aligned(A, es) && D % 4 == 0 && rot_dims % 4 == 0 && ldq % 4 == 0 && ((uintptr_t)q % (4 * es)) == 0 &&
                    ((uintptr_t)pages % (4 * es)) == 0;
-  const int V = vec && taps <= 4 ? 4 : 1;
+  const int V = vec && taps <= 4 ? 2 : 1;
   const long units = (long)(A.C / 2 / V);
   dim3 grid((unsigned)((units + CV_THREADS - 1) / CV_THREADS), R, (max_q_len + CV_TOKENS - 1) / CV_TOKENS);
 #define CVQ(TT, VV, MM) qe_launch(conv_qkv_kernel<TT, VV, MM>, grid, dim3(CV_THREADS), 0, stream, A, Q)
-#define CVQ_T(TT) do { if (taps > 4) CVQ(TT, 1, CV_MAX_TAPS); else if (V == 4) CVQ(TT, 4, 4); else CVQ(TT, 1, 4); } while (0)
+#define CVQ_T(TT) do { if (taps > 4) CVQ(TT, 1, CV_MAX_TAPS); else if (V == 2) CVQ(TT, 2, 4); else CVQ(TT, 1, 4); } while (0)
   if (dtype == QE_DTYPE_F32) CVQ_T(float); else CVQ_T(__nv_bfloat16);
 #undef CVQ_T
 #undef CVQ
